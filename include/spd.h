@@ -568,6 +568,9 @@ typedef struct {
   void* dst;
   int64_t src_row, dst_row;
   int32_t heads, head_dim, rot, src_head, dst_head, to_pool;
+  const float* norm_w;  /* norm != 0: after the bias and before the rotation the head is brought to unit RMS over its */
+  int32_t norm;         /* head_dim channels (norm_eps inside the root) and multiplied by norm_w (fp32 [head_dim], */
+  float norm_eps;       /* shared by the heads; NULL: no weight).  At most 512 channels then. */
 } spd_rotary_segment_t;
 /* Up to four segments in one launch.  cos_sin fp32 [max_positions, rot_max] = cos || sin (rot_max / 2 each) of
  * position * f_i; a segment with rot < rot_max uses the first rot / 2 of both.  paired != 0: channel 2 i turns
@@ -581,6 +584,71 @@ int spd_rotary_segments(const spd_rotary_segment_t* segments, int num_segments, 
 int spd_heads_gate(void* out, const void* a, const void* a2, const void* gate, int64_t tokens, int heads, int vdim,
                    int64_t a_stride, int64_t gate_stride, int64_t out_stride, float lambda, float eps, float post,
                    int dtype, spd_stream_t stream);
+
+/* ---------------------------------------------------------------------------------------------
+ * Layers that norm their sublayers' outputs, attention over a window and pooled blocks, recurrent
+ * mixers with one decay per head (csrc/mixer_ops.cu, attn_general*.cu, key_blocks.cuh, head_decay.cu)
+ * ------------------------------------------------------------------------------------------- */
+/* x[r, :] (fp32 [rows, dim], in place) += y[r, :] / sqrt(mean(y[r, :]^2) + eps) * coef (y dtype [rows, dim], coef fp32
+ * [dim]; both NULL: no update), then out[r, :] = x[r, :] in dtype or, with w [dim] given,
+ * x[r, :] / sqrt(mean(x[r, :]^2) + eps) * (weight_offset + w) (out NULL: update only). */
+int spd_residual_postnorm(void* out, float* x, const void* y, const float* coef, const void* w, int64_t rows,
+                          int64_t dim, float eps, float weight_offset, int dtype, spd_stream_t stream);
+/* x[i] = cap * tanh(x[i] / cap) for i < n */
+int spd_softcap_f32(float* x, int64_t n, float cap, spd_stream_t stream);
+/* spd_attn_general_ex over a window plus pooled blocks: besides its window, the query at position i sees one key and
+ * value for every block of block_size consecutive tokens of its request (block b: positions b * block_size ..) that
+ * lies wholly before the window, b * block_size + block_size - 1 <= i - window; tokens and blocks share one softmax.
+ * A block's row of k_pool / v_pool is block_base + run * ceil(block_run_len / block_size) + offset / block_size with
+ * run, offset the quotient and remainder of (slot of the block's last token - 1) by block_run_len: the cache hands out
+ * slots in runs of block_run_len consecutive positions.  block_size 0: no blocks.  Needs window > 0, slopes NULL. */
+int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const void* v_pool,
+                            const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
+                            const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                            int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                            int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
+                            float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
+                            int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
+                            int64_t v_slot_stride, int block_size, int block_run_len, int64_t block_base, int dtype,
+                            spd_stream_t stream);
+/* Writes the rows of the blocks that a batch's new tokens complete (their K / V are in the pool already): the mean over
+ * the block's token rows of k_pool (rows of k_row_elems) and v_pool (v_row_elems; v_pool NULL: keys only), summed in
+ * fp32.  Decode (seq_lens) or ragged extend (max_extend_len: host-side bound of extend_lens); slot 0 is padding. */
+int spd_pool_key_blocks(void* k_pool, void* v_pool, const int32_t* req_to_token, const int64_t* req_pool_indices,
+                        const int64_t* seq_lens, const int32_t* prefix_lens, const int32_t* extend_lens,
+                        int64_t batch, int64_t max_extend_len, int64_t req_to_token_stride, int64_t k_row_elems,
+                        int64_t v_row_elems, int block_size, int block_run_len, int64_t block_base, int dtype,
+                        spd_stream_t stream);
+/* Recurrence with one decay per head and token: dt = softplus(z + dt_bias), w = exp(-exp(a_log) dt); per head a matrix
+ * S (fp32, stored [v_dim][head_dim]) at slot req_pool_indices[r] of state [slots, heads, v_dim, head_dim] (zero for a
+ * request that starts at position 0), written back.  Head h uses key / query head h / (num_heads / num_k_heads).
+ *   form 0: S <- w S + dt k v^T;  o = S^T (q q_scale) + skip v                      (skip fp32 [heads], nullable)
+ *   form 1: k <- k / sqrt(sum k^2 + unit_eps), q <- q q_scale / sqrt(sum q^2 + unit_eps);  S <- w S;
+ *           u = sigmoid(b) (v - S^T k);  S <- S + k u^T;  o = S^T q
+ * q, k [tokens, num_k_heads * head_dim], v [tokens, num_heads * v_dim], z, b [tokens, num_heads] (dtype, row strides
+ * given; b read by form 1); dt_bias, a_log fp32 [heads].  head_dim <= 256.  Decode / ragged extend and padded rows as
+ * spd_retention.  o fp32 [tokens, num_heads * v_dim]. */
+int spd_head_decay(float* o, const void* q, const void* k, const void* v, const void* z, const void* b, float* state,
+                   const int64_t* req_pool_indices, const int64_t* seq_lens, const int64_t* out_cache_loc,
+                   const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                   int64_t batch, int num_heads, int num_k_heads, int head_dim, int v_dim, int64_t q_stride,
+                   int64_t k_stride, int64_t v_stride, int64_t z_stride, int64_t b_stride, const float* dt_bias,
+                   const float* a_log, const float* skip, int form, float q_scale, float unit_eps, int dtype,
+                   spd_stream_t stream);
+/* out[t, c] = silu(sum_{i < taps} w[i, c] x[t - (taps - 1) + i, c] + bias[c]) within each request (x rows of stride
+ * x_stride, w [taps, channels], bias nullable, out [total_rows, channels], all dtype).  The taps - 1 inputs before a
+ * request's first new row are conv_state[req_pool_indices[r]] (fp32 [slots, taps - 1, channels], oldest first; zeros at
+ * position 0), which then receives its last taps - 1 inputs.  taps <= 8.  max_rows_per_request: host-side bound of
+ * extend_lens (0: total_rows). */
+int spd_short_conv(void* out, const void* x, const void* w, const void* bias, float* conv_state,
+                   const int64_t* req_pool_indices, const int64_t* seq_lens, const int64_t* out_cache_loc,
+                   const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                   int64_t batch, int64_t total_rows, int64_t max_rows_per_request, int64_t channels, int taps,
+                   int64_t x_stride, int dtype, spd_stream_t stream);
+/* a = y silu(z); out = a / sqrt(mean(a^2) + eps) * w with the mean over each of `groups` equal parts of `part` channels
+ * (y fp32 [rows, groups * part], z rows of stride z_stride, w [groups * part]) */
+int spd_gated_group_norm(void* out, const float* y, const void* z, const void* w, int64_t rows, int groups, int part,
+                         int64_t z_stride, float eps, int dtype, spd_stream_t stream);
 
 #ifdef __cplusplus
 }

@@ -144,6 +144,21 @@ SIGNATURES = {
     "spd_residual_tanh_norm": (_i, [_p, _p, _p, _p, _p, _p, _p, _p, _i64, _i64, _f, _i, _p]),
     "spd_rotary_segments": (_i, [_p, _i, _p, _p, _p, _i, _i64, _i, _i64, _i, _p]),
     "spd_heads_gate": (_i, [_p, _p, _p, _p, _i64, _i, _i, _i64, _i64, _i64, _f, _f, _f, _i, _p]),
+    "spd_residual_postnorm": (_i, [_p, _p, _p, _p, _p, _i64, _i64, _f, _f, _i, _p]),
+    "spd_softcap_f32": (_i, [_p, _i64, _f, _p]),
+    "spd_attn_general_blocks": (
+        _i,
+        [_p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i64, _i64, _i, _i, _i, _i, _i64, _i64, _i64, _f, _i, _p, _p,
+         _f, _i, _i64, _f, _i, _i64, _i, _i, _i64, _i, _p],
+    ),
+    "spd_pool_key_blocks": (_i, [_p, _p, _p, _p, _p, _p, _p, _i64, _i64, _i64, _i64, _i64, _i, _i, _i64, _i, _p]),
+    "spd_head_decay": (
+        _i,
+        [_p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i64, _i, _i, _i, _i, _i64, _i64, _i64, _i64, _i64, _p, _p,
+         _p, _i, _f, _f, _i, _p],
+    ),
+    "spd_short_conv": (_i, [_p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i64, _i64, _i64, _i64, _i, _i64, _i, _p]),
+    "spd_gated_group_norm": (_i, [_p, _p, _p, _p, _i64, _i, _i, _i64, _f, _i, _p]),
     "spd_attn_prefill_simt": (
         _i,
         [_p, _p, _p, _p, _p, _p, _p, _p, _p, _i64, _i64, _i64, _i, _i, _i, _i64, _i64, _i64, _f, _i, _p],
@@ -159,7 +174,7 @@ class RotarySegment(C.Structure):
     """spd_rotary_segment_t of include/spd.h."""
     _fields_ = [("src", _p), ("bias", _p), ("dst", _p), ("src_row", _i64), ("dst_row", _i64), ("heads", C.c_int32),
                 ("head_dim", C.c_int32), ("rot", C.c_int32), ("src_head", C.c_int32), ("dst_head", C.c_int32),
-                ("to_pool", C.c_int32)]
+                ("to_pool", C.c_int32), ("norm_w", _p), ("norm", C.c_int32), ("norm_eps", _f)]
 
 
 def declared_functions(header_path: str = HEADER_PATH):

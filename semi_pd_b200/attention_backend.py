@@ -68,7 +68,7 @@ class RadixAttention:
                  sliding_window_size: int = -1, is_cross_attention: bool = False, prefix: str = "",
                  sinks: Optional[torch.Tensor] = None, distance_slopes: Optional[torch.Tensor] = None,
                  query_temperature: Optional[tuple] = None, general: bool = False, num_v_heads: int = 0,
-                 v_slot_stride: int = 0):
+                 v_slot_stride: int = 0, block_pool: int = 0):
         self.tp_q_head_num = num_heads
         self.tp_k_head_num = num_kv_heads
         self.tp_v_head_num = num_kv_heads
@@ -93,6 +93,9 @@ class RadixAttention:
         self.num_v_heads = num_v_heads or num_kv_heads
         self.v_slot_stride = v_slot_stride
         self.tp_v_head_num = self.num_v_heads
+        # also the general kernel's: tokens per pooled block; the tokens before the window are seen as one mean key and
+        # value per complete block of that many tokens (0: not at all).  Their rows belong to the layer's KV pool.
+        self.block_pool = int(block_pool)
         self.general = bool(general or sinks is not None or distance_slopes is not None or query_temperature
                             or self.sliding_window_size > 0 or self.v_head_dim != self.qk_head_dim)
         self.k_scale = None
@@ -177,6 +180,14 @@ class SpdAttnBackend(AttentionBackend):
                       sinks=layer.sinks, slopes=layer.distance_slopes, qtemp_coef=coef, qtemp_every=every,
                       softcap=layer.logit_cap, num_v_heads=layer.num_v_heads, v_slot_stride=layer.v_slot_stride)
         r2t = forward_batch.req_to_token_pool.req_to_token
+        if layer.block_pool:
+            pool = forward_batch.token_to_kv_pool
+            common["blocks"] = pool.get_blocks(layer.layer_id)
+            if pool.writes_blocks(layer.layer_id):  # the first layer over these keys with this block size
+                rows = self._batch_rows(forward_batch)
+                rows.pop("out_cache_loc", None), rows.pop("extend_start_loc", None)
+                ops.pool_key_blocks(k_buf, v_buf, r2t, forward_batch.req_pool_indices, common["blocks"],
+                                    max_extend_len=self.max_extend_len, **rows)
         if forward_batch.forward_mode.is_decode():
             return ops.attn_general(q, k_buf, v_buf, r2t, forward_batch.req_pool_indices,
                                     seq_lens=forward_batch.seq_lens, **common)
@@ -265,6 +276,26 @@ class SpdAttnBackend(AttentionBackend):
         if not forward_batch.forward_mode.is_decode():
             rows["max_extend_len"] = self.max_extend_len
         return ops.token_shift_mix(h, mu, shift, forward_batch.req_pool_indices, **rows)
+
+    def forward_short_conv(self, x, weight, bias, layer, forward_batch: ForwardBatch):
+        """Short causal convolution + SiLU of a mixer's projections: → [T, channels]; the taps − 1 inputs before a
+        request's first new row come from (and its last ones go to) the layer's vector state slot."""
+        rows = self._batch_rows(forward_batch)
+        if not forward_batch.forward_mode.is_decode():
+            rows["max_extend_len"] = self.max_extend_len
+        return ops.short_conv(x, weight, bias, forward_batch.token_to_kv_pool.state_pool.get_shift(layer.layer_id),
+                              forward_batch.req_pool_indices, **rows)
+
+    def forward_head_decay(self, q, k, v, z, layer, forward_batch: ForwardBatch, b=None):
+        """Recurrence with one decay per head over the request's state slot (stored [v_dim][head_dim] per head).  `layer`
+        carries num_heads, num_k_heads, head_dim, v_head_dim, layer_id, form ("ssd" | "delta"), q_scale, unit_eps,
+        dt_bias, a_log and skip (fp32 [heads]; skip None for "delta"); z and b are the raw step-size and write-strength
+        projections.  → o fp32 [T, heads · v_head_dim]."""
+        state = forward_batch.token_to_kv_pool.state_pool.get_state(layer.layer_id)
+        return ops.head_decay_recurrence(q, k, v, z, state, forward_batch.req_pool_indices, num_heads=layer.num_heads,
+                                         num_k_heads=layer.num_k_heads, head_dim=layer.head_dim, v_dim=layer.v_head_dim,
+                                         form=layer.form, dt_bias=layer.dt_bias, a_log=layer.a_log, skip=layer.skip, b=b,
+                                         q_scale=layer.q_scale, unit_eps=layer.unit_eps, **self._batch_rows(forward_batch))
 
     def forward_extend(self, q, k, v, layer: RadixAttention, forward_batch: ForwardBatch,
                        save_kv_cache: bool = True):

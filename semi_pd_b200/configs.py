@@ -78,6 +78,8 @@ class ModelConfig:
     embedding_scale: float = 1.0
     pair_embedding: Optional[dict] = None
     loop_times: int = 1
+    # model_type "fudonex": logits <- cap * tanh(logits / cap) (None: as they are)
+    logit_softcap: Optional[float] = None
 
     @property
     def context_len(self) -> int:
@@ -287,9 +289,69 @@ def _sugelix_config(path: str, cfg: dict, **overrides) -> ModelConfig:
     return ModelConfig(name=os.path.basename(os.path.normpath(path)) or "sugelix", **kw)
 
 
+_FUDONEX_MIXERS = ("attention", "mamba2", "delta")
+
+
+def _fudonex_config(path: str, cfg: dict, **overrides) -> ModelConfig:
+    """config.json of the Fudonex family: {"architecture", "vocab", "width", "norm": {"eps"}, "embedding": {"scale"},
+    "residual_mult", "logit_softcap", "layers": [{"type", "mixer", "mlp": {"kind": "dense", "ff"} | null}, ...]}.
+    Mixers: "attention" {heads, kv_heads, dim, vdim, scale, mask: {size, pool}, rot: {dims, base, scaling: {factor,
+    original, fast, slow}}, kv_from} (kv_from: an earlier attention layer whose cached keys and values are read), "mamba2"
+    {heads, vdim, state, groups, conv, norm_groups}, "delta" {heads, kv_heads, dim, vdim, conv}.  Every size and constant
+    is carried per layer in `layer_specs`."""
+    layers = [dict(spec) for spec in cfg["layers"]]
+    for i, spec in enumerate(layers):
+        if spec["type"] not in _FUDONEX_MIXERS:
+            raise ValueError(f"layer {i}: unknown mixer type {spec['type']!r}")
+        if spec.get("mlp") is not None and spec["mlp"].get("kind") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {spec['mlp'].get('kind')!r}")
+        m = spec["mixer"]
+        heads = int(m["heads"])
+        if spec["type"] == "mamba2":
+            if heads % int(m["groups"]) or (heads * int(m["vdim"])) % int(m["norm_groups"]):
+                raise ValueError(f"layer {i}: {heads} heads of {m['vdim']} do not split into {m['groups']} groups and "
+                                 f"{m['norm_groups']} norm groups")
+        elif heads % int(m.get("kv_heads", heads)):
+            raise ValueError(f"layer {i}: {heads} heads are not a multiple of {m['kv_heads']} kv heads")
+        if spec["type"] != "attention":
+            if int(m["conv"]) < 1:
+                raise ValueError(f"layer {i}: a convolution of {m['conv']} taps")
+            continue
+        rot, mask = int((m.get("rot") or {}).get("dims") or 0), m.get("mask") or {}
+        if rot % 2 or rot > int(m["dim"]):
+            raise ValueError(f"layer {i}: rot.dims {rot} must be even and at most dim {m['dim']}")
+        for key in ("size", "pool"):
+            if mask.get(key) is not None and int(mask[key]) < 1:
+                raise ValueError(f"layer {i}: mask.{key} {mask[key]} must be positive")
+        if mask.get("pool") is not None and mask.get("size") is None:
+            raise ValueError(f"layer {i}: pooled blocks need a window")
+        j = m.get("kv_from")
+        if j is not None:
+            if not 0 <= int(j) < i or layers[j]["type"] != "attention" or layers[j]["mixer"].get("kv_from") is not None:
+                raise ValueError(f"layer {i}: kv_from {j} must name an earlier attention layer with its own keys")
+            src = layers[j]["mixer"]
+            if any(int(m.get(k, m["heads"] if k == "kv_heads" else 0)) != int(src.get(k, src["heads"] if k == "kv_heads" else 0))
+                   for k in ("kv_heads", "dim", "vdim")):
+                raise ValueError(f"layer {i}: kv_heads, dim and vdim differ from layer {j}, whose keys it reads")
+    attn = [s["mixer"] for s in layers if s["type"] == "attention"]
+    cap = cfg.get("logit_softcap")
+    kw = dict(model_type="fudonex", hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]),
+              num_hidden_layers=len(layers), rms_norm_eps=float(cfg["norm"]["eps"]), layer_specs=layers,
+              embedding_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
+              residual_mult=float(cfg.get("residual_mult", 1.0)), logit_softcap=float(cap) if cap else None,
+              tie_word_embeddings=True,
+              # summary fields other components print or size by; the per-layer values rule
+              num_attention_heads=max([int(m["heads"]) for m in attn] or [1]),
+              num_key_value_heads=max([int(m.get("kv_heads", m["heads"])) for m in attn] or [1]),
+              head_dim=max([int(m["dim"]) for m in attn] or [1]), intermediate_size=0,
+              max_position_embeddings=int(cfg.get("context", 8192)))
+    kw.update(overrides)
+    return ModelConfig(name=os.path.basename(os.path.normpath(path)) or "fudonex", **kw)
+
+
 # config.json "architecture" -> reader
 _ARCHITECTURE_READERS = {"Rimidra": _rimidra_config, "Nupovik": _nupovik_config, "Matepel": _matepel_config,
-                         "Sugelix": _sugelix_config}
+                         "Sugelix": _sugelix_config, "Fudonex": _fudonex_config}
 
 
 def load_model_config(path: str, **overrides) -> ModelConfig:

@@ -1,6 +1,7 @@
 // Softmax attention over the paged KV pool with the options the tcgen05 kernels do not have:
 // a sliding window, a learned per-head sink in the denominator, a linear distance bias, a
-// position-dependent query temperature, key size != value size, and 32-bit storage.  Decode and
+// position-dependent query temperature, key size != value size, pooled blocks of the tokens that lie
+// before the window (key_blocks.cuh), and 32-bit storage.  Decode and
 // ragged extend (chunked prefill, mixed batches) are the same kernel: one warp owns one (query
 // token, query head), walks its visible keys in tiles of 32 (one key per lane for the scores, one
 // slice of the value row per lane for the output) and keeps the online-softmax state in fp32.
@@ -8,6 +9,7 @@
 // Beside attn_simt.cu (plain causal SIMT attention) in role; the reference has no such kernel.
 #include "common.cuh"
 #include "ptx.cuh"
+#include "key_blocks.cuh"
 #include <stdlib.h>
 
 namespace spd {
@@ -60,7 +62,7 @@ attn_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __res
                     const int32_t* __restrict__ extend_start_loc, int batch, int64_t total_tokens, int H, int G,
                     int dk, int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale,
                     int window, const float* __restrict__ sinks, const float* __restrict__ slopes, float qtemp_coef,
-                    int qtemp_every, float softcap, int Gv, int64_t v_slot) {
+                    int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
   extern __shared__ float q_smem[];  // [4][dk]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   // item = h * tokens_padded + t with tokens_padded a multiple of 4: the warps of a CTA share a head
@@ -104,16 +106,17 @@ attn_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __res
   for (int i = 0; i < VMAX; ++i) acc[i] = 0.f;
 
   const int64_t j_lo = window > 0 ? (pos - window + 1 > 0 ? pos - window + 1 : 0) : 0;
-  for (int64_t j0 = j_lo; j0 <= pos; j0 += 32) {
-    const int64_t j = j0 + lane;
-    const bool valid = j <= pos;
+  const int64_t nb = key_blocks_seen(kb, pos, window), n_keys = nb + pos - j_lo + 1;  // blocks, then tokens
+  for (int64_t e0 = 0; e0 < n_keys; e0 += 32) {
+    const int64_t e = e0 + lane;
+    const bool valid = e < n_keys;
     int slot = 0;
     float s = -INFINITY;
     if (valid) {
-      slot = page[j];
+      slot = key_row(kb, page, e, nb, j_lo);
       s = dot_row<T>(qs, k_pool + ((int64_t)slot * G + g) * dk, dk);
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-      s -= slope * (float)(pos - j);
+      s -= slope * (float)(n_keys - 1 - e);  // distance of a token (blocks come without a slope)
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);  // m = -inf (first tile, no sink): 0
@@ -122,7 +125,7 @@ attn_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __res
     m = m_new;
 #pragma unroll
     for (int i = 0; i < VMAX; ++i) acc[i] *= corr;
-    const int n = (int)(pos - j0 + 1 < 32 ? pos - j0 + 1 : 32);
+    const int n = (int)(n_keys - e0 < 32 ? n_keys - e0 : 32);
     for (int jj = 0; jj < n; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const int sj = __shfl_sync(0xffffffffu, slot, jj);
@@ -153,7 +156,7 @@ attn_general_decode_kernel(T* __restrict__ out, const T* __restrict__ q, const T
                            int G, int dk, int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride,
                            float sm_scale, int window, const float* __restrict__ sinks,
                            const float* __restrict__ slopes, float qtemp_coef, int qtemp_every, float softcap, int Gv,
-                           int64_t v_slot) {
+                           int64_t v_slot, KeyBlocks kb) {
   extern __shared__ float dec_smem[];  // q [dk] | m [4] | l [4] | acc [4][dv]
   float* qs = dec_smem;
   float* sm_m = qs + dk;
@@ -176,16 +179,17 @@ attn_general_decode_kernel(T* __restrict__ out, const T* __restrict__ q, const T
 #pragma unroll
   for (int i = 0; i < VMAX; ++i) acc[i] = 0.f;
   const int64_t j_lo = window > 0 ? (pos - window + 1 > 0 ? pos - window + 1 : 0) : 0;
-  for (int64_t j0 = j_lo + 32 * warp; j0 <= pos; j0 += 128) {
-    const int64_t j = j0 + lane;
-    const bool valid = j <= pos;
+  const int64_t nb = key_blocks_seen(kb, pos, window), n_keys = nb + pos - j_lo + 1;  // blocks, then tokens
+  for (int64_t e0 = 32 * warp; e0 < n_keys; e0 += 128) {
+    const int64_t e = e0 + lane;
+    const bool valid = e < n_keys;
     int slot = 0;
     float s = -INFINITY;
     if (valid) {
-      slot = page[j];
+      slot = key_row(kb, page, e, nb, j_lo);
       s = dot_row<T>(qs, k_pool + ((int64_t)slot * G + g) * dk, dk);
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-      s -= slope * (float)(pos - j);
+      s -= slope * (float)(n_keys - 1 - e);  // distance of a token (blocks come without a slope)
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);
@@ -194,7 +198,7 @@ attn_general_decode_kernel(T* __restrict__ out, const T* __restrict__ q, const T
     m = m_new;
 #pragma unroll
     for (int i = 0; i < VMAX; ++i) acc[i] *= corr;
-    const int n = (int)(pos - j0 + 1 < 32 ? pos - j0 + 1 : 32);
+    const int n = (int)(n_keys - e0 < 32 ? n_keys - e0 : 32);
     for (int jj = 0; jj < n; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const int sj = __shfl_sync(0xffffffffu, slot, jj);
@@ -284,7 +288,7 @@ attn_general_decode_group_kernel(T* __restrict__ out, const T* __restrict__ q, c
                                  int H, int G, int dk, int64_t q_stride, int64_t out_stride, int64_t r2t_stride,
                                  float sm_scale, int window, const float* __restrict__ sinks,
                                  const float* __restrict__ slopes, float qtemp_coef, int qtemp_every, int q_bytes,
-                                 float softcap, int Gv, int64_t v_slot) {
+                                 float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
   constexpr int N = 16 / (int)sizeof(T);
   constexpr int DV = 32 * VPL;
   constexpr int vstride = DV * (int)sizeof(T) + 16;
@@ -323,11 +327,12 @@ attn_general_decode_group_kernel(T* __restrict__ out, const T* __restrict__ q, c
   constexpr int v_rows = vc >= 32 ? 1 : 32 / vc;
   const int v_lrow = vc >= 32 ? 0 : lane / vc, v_lch = vc >= 32 ? lane : lane - v_lrow * vc;
   const int64_t j_lo = window > 0 ? (pos - window + 1 > 0 ? pos - window + 1 : 0) : 0;
-  for (int64_t j0 = j_lo + 32 * warp; j0 <= pos; j0 += 32 * NW) {
-    const int n = (int)(pos - j0 + 1 < 32 ? pos - j0 + 1 : 32);
+  const int64_t nb = key_blocks_seen(kb, pos, window), n_keys = nb + pos - j_lo + 1;  // blocks, then tokens
+  for (int64_t e0 = 32 * warp; e0 < n_keys; e0 += 32 * NW) {
+    const int n = (int)(n_keys - e0 < 32 ? n_keys - e0 : 32);
     const bool valid = lane < n;
     __syncwarp();  // the previous tile has been read
-    if (valid) slots[lane] = page[j0 + lane];
+    if (valid) slots[lane] = key_row(kb, page, e0 + lane, nb, j_lo);
     __syncwarp();
     if (lane < k_rows * kc)
       for (int kk = k_lrow; kk < n; kk += k_rows) {
@@ -368,7 +373,7 @@ attn_general_decode_group_kernel(T* __restrict__ out, const T* __restrict__ q, c
         }
       }
     }
-    const float dist = (float)(pos - (j0 + lane));
+    const float dist = (float)(n_keys - 1 - (e0 + lane));
     float p[RMAX];
 #pragma unroll
     for (int rr = 0; rr < RMAX; ++rr) {
@@ -442,7 +447,7 @@ int attn_general_decode_group_launch(size_t smem, int q_bytes, int64_t batch, cu
                                      const int64_t* req_pool_indices, const int64_t* seq_lens, int H, int G, int dk,
                                      int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                                      const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every,
-                                     float softcap, int Gv, int64_t v_slot) {
+                                     float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
     SPD_CUDA(cudaFuncSetAttribute(attn_general_decode_group_kernel<T, VPL, RMAX, NW>,
@@ -452,7 +457,7 @@ int attn_general_decode_group_launch(size_t smem, int q_bytes, int64_t batch, cu
   SPD_CUDA(launch(attn_general_decode_group_kernel<T, VPL, RMAX, NW>, dim3((unsigned)batch, (unsigned)G), dim3(NW * 32), smem,
                   stream, /*pdl=*/false, (T*)out, (const T*)q, (const T*)k_pool, (const T*)v_pool, req_to_token,
                   req_pool_indices, seq_lens, H, G, dk, q_stride, out_stride, r2t_stride, sm_scale, window, sinks, slopes,
-                  qtemp_coef, qtemp_every, q_bytes, softcap, Gv, v_slot));
+                  qtemp_coef, qtemp_every, q_bytes, softcap, Gv, v_slot, kb));
   return 0;
 }
 
@@ -467,19 +472,70 @@ kv_store_kernel(const T* __restrict__ k, const T* __restrict__ v, T* __restrict_
     for (int64_t i = threadIdx.x; i < v_row; i += 256) v_pool[slot * v_row + i] = v[t * v_stride + i];
 }
 
+// Block rows of the blocks that a batch completes: the mean over the block's cache rows of K and V, as the cache holds
+// them, in fp32.  One CTA per (request, block that its new tokens may complete).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128)
+pool_key_blocks_kernel(T* __restrict__ k_pool, T* __restrict__ v_pool, const int32_t* __restrict__ req_to_token,
+                       const int64_t* __restrict__ req_pool_indices, const int64_t* __restrict__ seq_lens,
+                       const int32_t* __restrict__ prefix_lens, const int32_t* __restrict__ extend_lens,
+                       int64_t r2t_stride, int64_t k_row, int64_t v_row, KeyBlocks kb) {
+  griddep_wait();
+  griddep_launch_dependents();
+  const int r = blockIdx.y;
+  const int64_t pos0 = seq_lens != nullptr ? seq_lens[r] - 1 : (int64_t)prefix_lens[r];
+  const int64_t end = seq_lens != nullptr ? pos0 + 1 : pos0 + extend_lens[r];  // tokens cached by now
+  if (pos0 < 0) return;
+  const int64_t first = (pos0 / kb.size + blockIdx.x) * kb.size;
+  if (first + kb.size > end) return;
+  const int32_t* page = req_to_token + req_pool_indices[r] * r2t_stride + first;
+  if (page[kb.size - 1] <= 0) return;  // a padded row of a captured batch
+  const int64_t row = key_block_row(kb, page[kb.size - 1]);
+  const float inv = 1.0f / (float)kb.size;
+  auto mean = [&](T* pool, int64_t n) {
+    for (int64_t c = threadIdx.x * VEC; c < n; c += 128 * VEC) {
+      float acc[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+#pragma unroll 4
+      for (int i = 0; i < kb.size; ++i) {
+        const T* src = pool + (int64_t)page[i] * n + c;
+        if constexpr (VEC == 1) {
+          acc[0] += to_f32<T>(src[0]);
+        } else {
+          const Vec16<T> x = ldv(src);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) acc[e] += to_f32<T>(x.e()[e]);
+        }
+      }
+      T* dst = pool + row * n + c;
+      if constexpr (VEC == 1) {
+        dst[0] = from_f32<T>(acc[0] * inv);
+      } else {
+        Vec16<T> x;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x.e()[e] = from_f32<T>(acc[e] * inv);
+        stv(dst, x);
+      }
+    }
+  };
+  mean(k_pool, k_row);
+  if (v_pool != nullptr) mean(v_pool, v_row);
+}
+
 int attn_general_mma_try(void* out, const void* q, const void* k_pool, const void* v_pool, const int32_t* req_to_token,
                          const int64_t* req_pool_indices, const int32_t* prefix_lens, const int32_t* extend_lens,
                          const int32_t* extend_start_loc, int64_t batch, int64_t max_extend_len, int H, int G, int dk,
                          int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                          const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap,
-                         int Gv, int64_t v_slot, int dtype, cudaStream_t stream);
+                         int Gv, int64_t v_slot, KeyBlocks kb, int dtype, cudaStream_t stream);
 
 int attn_general_mma_decode_try(void* out, const void* q, const void* k_pool, const void* v_pool,
                                 const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
                                 int64_t batch, int H, int G, int dk, int dv, int64_t q_stride, int64_t out_stride,
                                 int64_t r2t_stride, float sm_scale, int window, const float* sinks, const float* slopes,
-                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, int dtype,
-                                cudaStream_t stream);
+                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb,
+                                int dtype, cudaStream_t stream);
 
 }  // namespace spd
 
@@ -501,20 +557,50 @@ int spd_kv_store(const void* k, const void* v, void* k_pool, void* v_pool, const
   return 0;
 }
 
-int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void* v_pool,
-                        const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
-                        const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
-                        int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
-                        int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
-                        float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
-                        int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
-                        int64_t v_slot_stride, int dtype, spd_stream_t stream) {
+int spd_pool_key_blocks(void* k_pool, void* v_pool, const int32_t* req_to_token, const int64_t* req_pool_indices,
+                        const int64_t* seq_lens, const int32_t* prefix_lens, const int32_t* extend_lens, int64_t batch,
+                        int64_t max_extend_len, int64_t req_to_token_stride, int64_t k_row_elems, int64_t v_row_elems,
+                        int block_size, int block_run_len, int64_t block_base, int dtype, spd_stream_t stream) {
+  SPD_REQUIRE(k_pool && req_to_token && req_pool_indices, SPD_E_BADARG, "spd_pool_key_blocks: null pointer");
+  SPD_REQUIRE(seq_lens != nullptr || (prefix_lens && extend_lens), SPD_E_BADARG,
+              "spd_pool_key_blocks: extend needs prefix_lens and extend_lens");
+  SPD_REQUIRE(block_size > 0 && block_run_len > 0 && block_base > 0 && k_row_elems > 0 && v_row_elems >= 0, SPD_E_BADARG,
+              "spd_pool_key_blocks: bad sizes");
+  const int64_t rows = seq_lens != nullptr ? 1 : max_extend_len;
+  if (batch == 0 || rows <= 0) return 0;
+  SPD_REQUIRE(batch <= 65535, SPD_E_SHAPE, "spd_pool_key_blocks: batch too large");
+  const KeyBlocks kb{block_size, block_run_len, (block_run_len + block_size - 1) / block_size, block_base};
+  const dim3 grid((unsigned)((rows + block_size - 1) / block_size), (unsigned)batch);  // n new tokens complete at most that many
+  SPD_DISPATCH_ANY(dtype, {
+    constexpr int N = 16 / (int)sizeof(T);
+    const bool vec = k_row_elems % N == 0 && v_row_elems % N == 0 && aligned16(k_pool) && aligned16(v_pool);
+    auto kern = vec ? pool_key_blocks_kernel<T, N> : pool_key_blocks_kernel<T, 1>;
+    SPD_CUDA(launch(kern, grid, dim3(128), 0, as_stream(stream), pdl_enabled(), (T*)k_pool, (T*)v_pool, req_to_token,
+                    req_pool_indices, seq_lens, prefix_lens, extend_lens, req_to_token_stride, k_row_elems, v_row_elems,
+                    kb));
+  });
+  return 0;
+}
+
+int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const void* v_pool,
+                            const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
+                            const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                            int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                            int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
+                            float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
+                            int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
+                            int64_t v_slot_stride, int block_size, int block_run_len,
+                                int64_t block_base, int dtype, spd_stream_t stream) {
   if (num_v_heads <= 0) num_v_heads = num_kv_heads;
   if (v_slot_stride <= 0) v_slot_stride = (int64_t)num_v_heads * v_dim;
   const int Gv = num_v_heads;
   const int64_t v_slot = v_slot_stride;
   SPD_REQUIRE(num_kv_heads % num_v_heads == 0 && softcap >= 0.f, SPD_E_SHAPE,
               "spd_attn_general: kv heads %d not a multiple of value heads %d", num_kv_heads, num_v_heads);
+  SPD_REQUIRE(block_size == 0 || (block_size > 0 && block_run_len > 0 && block_base > 0 && window > 0 && slopes == nullptr),
+              SPD_E_BADARG, "spd_attn_general: pooled blocks need a window, a run length and a base row, and no distance bias");
+  const KeyBlocks kb{block_size, block_run_len, block_size > 0 ? (block_run_len + block_size - 1) / block_size : 0,
+                     block_base};
   SPD_REQUIRE(out && q && k_pool && v_pool && req_to_token && req_pool_indices, SPD_E_BADARG,
               "spd_attn_general: null pointer");
   SPD_REQUIRE(seq_lens != nullptr || (prefix_lens && extend_lens && extend_start_loc), SPD_E_BADARG,
@@ -532,7 +618,7 @@ int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void
       const int rc = attn_general_mma_decode_try(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, batch,
                                                  num_q_heads, num_kv_heads, head_dim, v_dim, q_stride, out_stride,
                                                  req_to_token_stride, sm_scale, window, sinks, slopes, qtemp_coef,
-                                                 qtemp_every, softcap, Gv, v_slot, dtype, as_stream(stream));
+                                                 qtemp_every, softcap, Gv, v_slot, kb, dtype, as_stream(stream));
       if (rc != 1) return rc;
     }
     // grouped form: 16-byte rows, v_dim 32 x {1, 2, 4, 8}, up to 8 query heads per key/value head
@@ -552,7 +638,7 @@ int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void
 #define SPD_GRP_ARGS                                                                                                  \
   gsmem, q_bytes, batch, as_stream(stream), out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens,         \
       num_q_heads, num_kv_heads, head_dim, q_stride, out_stride, req_to_token_stride, sm_scale, window, sinks, slopes, \
-      qtemp_coef, qtemp_every, softcap, Gv, v_slot
+      qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb
 #define SPD_GRP_R(TT, VPL)                                                                     \
   do {                                                                                         \
     if (R <= 1) return nw == 8 ? attn_general_decode_group_launch<TT, VPL, 1, 8>(SPD_GRP_ARGS)  \
@@ -584,7 +670,7 @@ int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void
                       as_stream(stream), /*pdl=*/false, (T*)out, (const T*)q, (const T*)k_pool, (const T*)v_pool,
                       req_to_token, req_pool_indices, seq_lens, num_q_heads, num_kv_heads, head_dim, v_dim, q_stride,
                       out_stride, req_to_token_stride, sm_scale, window, sinks, slopes, qtemp_coef, qtemp_every, softcap,
-                      Gv, v_slot));
+                      Gv, v_slot, kb));
     });
     return 0;
   }
@@ -592,7 +678,7 @@ int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void
     const int rc = attn_general_mma_try(out, q, k_pool, v_pool, req_to_token, req_pool_indices, prefix_lens, extend_lens,
                                         extend_start_loc, batch, max_extend_len, num_q_heads, num_kv_heads, head_dim,
                                         v_dim, q_stride, out_stride, req_to_token_stride, sm_scale, window, sinks, slopes,
-                                        qtemp_coef, qtemp_every, softcap, Gv, v_slot, dtype, as_stream(stream));
+                                        qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, dtype, as_stream(stream));
     if (rc != 1) return rc;
   }
   const int64_t tokens4 = (total_tokens + 3) / 4 * 4;
@@ -605,9 +691,24 @@ int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void
                     (T*)out, (const T*)q, (const T*)k_pool, (const T*)v_pool, req_to_token, req_pool_indices, seq_lens,
                     prefix_lens, extend_lens, extend_start_loc, (int)batch, total_tokens, num_q_heads, num_kv_heads,
                     head_dim, v_dim, q_stride, out_stride, req_to_token_stride, sm_scale, window, sinks, slopes,
-                    qtemp_coef, qtemp_every, softcap, Gv, v_slot));
+                    qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb));
   });
   return 0;
+}
+
+int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void* v_pool,
+                        const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
+                        const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                        int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                        int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
+                        float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
+                        int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
+                        int64_t v_slot_stride, int dtype, spd_stream_t stream) {
+    return spd_attn_general_blocks(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, prefix_lens,
+                                 extend_lens, extend_start_loc, batch, total_tokens, num_q_heads, num_kv_heads,
+                                 head_dim, v_dim, q_stride, out_stride, req_to_token_stride, sm_scale, window, sinks,
+                                 slopes, qtemp_coef, qtemp_every, max_extend_len, softcap, num_v_heads, v_slot_stride,
+                                 0, 0, 0, dtype, stream);
 }
 
 int spd_attn_general(void* out, const void* q, const void* k_pool, const void* v_pool,

@@ -4,11 +4,12 @@
 // table with 16-byte cp.async into a double-buffered shared-memory ring, S = Q K^T and O += P V run
 // on warp-level mma.sync.m16n8k16 (fp32 accumulators), and the online softmax — scale, temperature,
 // bias, window mask, sink — is fp32 in the exp2 domain.  Only the keys a tile can see are visited:
-// [first row - window + 1, last row].  The CUDA-core kernel of attn_general.cu keeps decode, float32
+// [first row - window + 1, last row], preceded by the pooled blocks it can see.  The CUDA-core kernel of attn_general.cu keeps decode, float32
 // models and head sizes outside the instantiated set.  (mma.sync, not tcgen05: the first tensor-core
 // kernel of this mechanism.)
 #include "common.cuh"
 #include "ptx.cuh"
+#include "key_blocks.cuh"
 #include <stdlib.h>
 
 namespace spd {
@@ -58,7 +59,7 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
                         const int32_t* __restrict__ extend_lens, const int32_t* __restrict__ extend_start_loc, int H,
                         int G, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                         const float* __restrict__ sinks, const float* __restrict__ slopes, float qtemp_coef,
-                        int qtemp_every, float softcap, int Gv, int64_t v_slot) {
+                        int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
   constexpr int LDK = DK + 8, LDV = DV + 8;  // +16 B per row: ldmatrix rows fall into distinct banks
   extern __shared__ __align__(16) unsigned char gm_smem[];
   T* sQ = reinterpret_cast<T*>(gm_smem);   // [BQ][LDK]
@@ -82,19 +83,21 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
   }
   const int64_t j_hi = i0 + nq - 1;
   const int64_t j_lo = window > 0 ? (i0 - window + 1 > 0 ? i0 - window + 1 : 0) : 0;
-  const int ntiles = (int)((j_hi - j_lo) / kGmBK) + 1;
+  // the tile's keys in one list: the NB blocks its last row sees, then the tokens j_lo .. j_hi
+  const int NB = (int)key_blocks_seen(kb, j_hi, window), n_keys = NB + (int)(j_hi - j_lo) + 1;
+  const int ntiles = (n_keys - 1) / kGmBK + 1;
   auto load_kv = [&](int t, int buf) {
-    const int64_t jb = j_lo + (int64_t)t * kGmBK;
+    const int eb = t * kGmBK;
     for (int idx = tid; idx < kGmBK * (DK / 8); idx += kGmThreads) {
       const int row = idx / (DK / 8), c = idx % (DK / 8);
-      const bool ok = jb + row <= j_hi;
-      const int64_t slot = ok ? page[jb + row] : 0;
+      const bool ok = eb + row < n_keys;
+      const int64_t slot = ok ? key_row(kb, page, eb + row, NB, j_lo) : 0;
       cp_async16(smem_u32(sK + (buf * kGmBK + row) * LDK + c * 8), k_pool + (slot * G + g) * DK + c * 8, ok);
     }
     for (int idx = tid; idx < kGmBK * (DV / 8); idx += kGmThreads) {
       const int row = idx / (DV / 8), c = idx % (DV / 8);
-      const bool ok = jb + row <= j_hi;
-      const int64_t slot = ok ? page[jb + row] : 0;
+      const bool ok = eb + row < n_keys;
+      const int64_t slot = ok ? key_row(kb, page, eb + row, NB, j_lo) : 0;
       cp_async16(smem_u32(sV + (buf * kGmBK + row) * LDV + c * 8), v_pool + slot * v_slot + (int64_t)(g % Gv) * DV + c * 8, ok);
     }
   };
@@ -103,6 +106,15 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
 
   const int rl[2] = {warp * 16 + (lane >> 2), warp * 16 + (lane >> 2) + 8};
   const int64_t pi[2] = {i0 + rl[0], i0 + rl[1]};
+  // what a row sees of the list: blocks [0, nbx), tokens [lo, hi] (nothing for rows past the portion)
+  int nbx[2], lo[2], hi[2];
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const bool ok = pi[x] <= j_hi;
+    nbx[x] = ok ? (int)key_blocks_seen(kb, pi[x], window) : 0;
+    hi[x] = ok ? NB + (int)(pi[x] - j_lo) : -1;
+    lo[x] = window > 0 && pi[x] - window + 1 > j_lo ? NB + (int)(pi[x] - window + 1 - j_lo) : NB;
+  }
   float sc[2], scc[2];  // score multipliers into the exp2 domain, and (with a cap) into units of the cap
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
@@ -148,18 +160,17 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
         gm_mma<T>(s[2 * nb2 + 1], a, b[2], b[3]);
       }
     }
-    const int64_t jb = j_lo + (int64_t)t * kGmBK;
+    const int eb = t * kGmBK;
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nb = 0; nb < kGmBK / 8; ++nb)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int x = e >> 1;
-        const int64_t j = jb + nb * 8 + (lane & 3) * 2 + (e & 1);
-        const int64_t dist = pi[x] - j;
-        const bool ok = dist >= 0 && (window <= 0 || dist < window) && pi[x] <= j_hi;
+        const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
+        const bool ok = (idx >= lo[x] && idx <= hi[x]) || idx < nbx[x];
         const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc[x]) : s[nb][e] * sc[x];
-        const float v = ok ? z - sl * (float)dist : -INFINITY;
+        const float v = ok ? z - sl * (float)(hi[x] - idx) : -INFINITY;
         s[nb][e] = v;
         mx[x] = fmaxf(mx[x], v);
       }
@@ -226,7 +237,7 @@ static int gm_launch(void* out, const void* q, const void* k_pool, const void* v
                      const int32_t* extend_start_loc, int64_t batch, int64_t max_extend_len, int H, int G,
                      int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                      const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap, int Gv,
-                     int64_t v_slot, cudaStream_t stream) {
+                     int64_t v_slot, KeyBlocks kb, cudaStream_t stream) {
   constexpr size_t smem = sizeof(T) * ((size_t)kGmBQ * (DK + 8) + 2 * kGmBK * (DK + 8) + 2 * kGmBK * (DV + 8));
   static bool configured = false;  // per instantiation
   if (!configured) {
@@ -237,7 +248,7 @@ static int gm_launch(void* out, const void* q, const void* k_pool, const void* v
   SPD_CUDA(launch(attn_general_mma_kernel<T, DK, DV>, grid, dim3(kGmThreads), smem, stream, /*pdl=*/false, (T*)out,
                   (const T*)q, (const T*)k_pool, (const T*)v_pool, req_to_token, req_pool_indices, prefix_lens,
                   extend_lens, extend_start_loc, H, G, q_stride, out_stride, r2t_stride, sm_scale, window, sinks, slopes,
-                  qtemp_coef, qtemp_every, softcap, Gv, v_slot));
+                  qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb));
   return 0;
 }
 
@@ -247,7 +258,7 @@ int attn_general_mma_try(void* out, const void* q, const void* k_pool, const voi
                          const int32_t* extend_start_loc, int64_t batch, int64_t max_extend_len, int H, int G, int dk,
                          int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                          const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap,
-                         int Gv, int64_t v_slot, int dtype, cudaStream_t stream) {
+                         int Gv, int64_t v_slot, KeyBlocks kb, int dtype, cudaStream_t stream) {
   if (dtype != SPD_BF16 && dtype != SPD_F16) return 1;
   if (v_slot % 8 != 0) return 1;
   if (max_extend_len < 16 || batch > 65535 || H > 65535) return 1;  // short portions: the CUDA-core kernel
@@ -260,11 +271,11 @@ int attn_general_mma_try(void* out, const void* q, const void* k_pool, const voi
       return gm_launch<__nv_bfloat16, DKV, DVV>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, prefix_lens, \
                                                 extend_lens, extend_start_loc, batch, max_extend_len, H, G, q_stride, \
                                                 out_stride, r2t_stride, sm_scale, window, sinks, slopes, qtemp_coef, \
-                                                qtemp_every, softcap, Gv, v_slot, stream);                          \
+                                                qtemp_every, softcap, Gv, v_slot, kb, stream);                          \
     return gm_launch<__half, DKV, DVV>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, prefix_lens,        \
                                        extend_lens, extend_start_loc, batch, max_extend_len, H, G, q_stride,        \
                                        out_stride, r2t_stride, sm_scale, window, sinks, slopes, qtemp_coef,         \
-                                       qtemp_every, softcap, Gv, v_slot, stream);                                   \
+                                       qtemp_every, softcap, Gv, v_slot, kb, stream);                                   \
   }
   SPD_GM_CASE(32, 32)
   SPD_GM_CASE(64, 64)
@@ -300,7 +311,7 @@ attn_general_mma_decode_kernel(T* __restrict__ out, const T* __restrict__ q, con
                                const int64_t* __restrict__ req_pool_indices, const int64_t* __restrict__ seq_lens,
                                int H, int G, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale,
                                int window, const float* __restrict__ sinks, const float* __restrict__ slopes,
-                               float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot) {
+                               float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
   constexpr int LDK = DK + 8, LDV = DV + 8;
   constexpr size_t kQBytes = sizeof(T) * 16 * LDK;
   constexpr size_t kWarpBytes = kGdWarpHdr + sizeof(T) * kGdTK * (LDK + LDV);
@@ -345,10 +356,11 @@ attn_general_mma_decode_kernel(T* __restrict__ out, const T* __restrict__ q, con
   constexpr int kc = DK / 8, vc = DV / 8;  // 16-byte chunks per row; vc divides 32, kc is at most 32
   const int64_t j_lo = window > 0 ? (pos - window + 1 > 0 ? pos - window + 1 : 0) : 0;
   const int n_split = gridDim.z;  // CTAs of the cluster that share this (request, head)
-  for (int64_t j0 = j_lo + kGdTK * ((int64_t)blockIdx.z * NW + warp); j0 <= pos; j0 += (int64_t)kGdTK * NW * n_split) {
-    const int n = (int)(pos - j0 + 1 < kGdTK ? pos - j0 + 1 : kGdTK);
+  const int64_t nblk = key_blocks_seen(kb, pos, window), n_keys = nblk + pos - j_lo + 1;  // blocks, then tokens
+  for (int64_t e0 = kGdTK * ((int64_t)blockIdx.z * NW + warp); e0 < n_keys; e0 += (int64_t)kGdTK * NW * n_split) {
+    const int n = (int)(n_keys - e0 < kGdTK ? n_keys - e0 : kGdTK);
     __syncwarp();  // the previous tile has been read
-    if (lane < n) slots[lane] = page[j0 + lane];
+    if (lane < n) slots[lane] = key_row(kb, page, e0 + lane, nblk, j_lo);
     __syncwarp();
     for (int row = lane / kc; row < kGdTK && lane < (32 / kc) * kc; row += 32 / kc) {  // (lanes past the last whole row idle)
       const bool ok = row < n;
@@ -389,7 +401,7 @@ attn_general_mma_decode_kernel(T* __restrict__ out, const T* __restrict__ q, con
         const int x = e >> 1;
         const int col = nb * 8 + (lane & 3) * 2 + (e & 1);
         const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc) : s[nb][e] * sc;
-        const float v = col < n ? z - sl[x] * (float)(pos - (j0 + col)) : -INFINITY;
+        const float v = col < n ? z - sl[x] * (float)(n_keys - 1 - (e0 + col)) : -INFINITY;
         s[nb][e] = v;
         mx[x] = fmaxf(mx[x], v);
       }
@@ -527,7 +539,7 @@ static int gd_launch_nw(void* out, const void* q, const void* k_pool, const void
                         const int64_t* req_pool_indices, const int64_t* seq_lens, int64_t batch, int H, int G,
                         int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                         const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap, int Gv,
-                        int64_t v_slot, cudaStream_t stream) {
+                        int64_t v_slot, KeyBlocks kb, cudaStream_t stream) {
   constexpr size_t tiles = (size_t)NW * (kGdWarpHdr + sizeof(T) * kGdTK * (DK + 8 + DV + 8));
   constexpr size_t merge = sizeof(float) * (NW + 1) * 16 * (DV + 2);  // the warps' triples + the CTA's own
   constexpr size_t smem = sizeof(T) * 16 * (DK + 8) + (tiles > merge ? tiles : merge);
@@ -542,7 +554,7 @@ static int gd_launch_nw(void* out, const void* q, const void* k_pool, const void
   int split = 1;
   const int64_t pairs = batch * G * ((H / G + 15) / 16);
   const int sms = device_sm_count_cached();
-  const int64_t max_split = window > 0 ? (window + kGdTK * NW - 1) / (kGdTK * NW) : 8;
+  const int64_t max_split = window > 0 && kb.size == 0 ? (window + kGdTK * NW - 1) / (kGdTK * NW) : 8;
   while (split * 2 <= 8 && split * 2 <= max_split && pairs * split * 2 <= sms) split *= 2;
   static const bool no_split = getenv("SPD_ATTN_DECODE_NO_SPLIT") != nullptr;
   if (no_split) split = 1;
@@ -561,7 +573,7 @@ static int gd_launch_nw(void* out, const void* q, const void* k_pool, const void
   SPD_CUDA(cudaLaunchKernelEx(&cfg, attn_general_mma_decode_kernel<T, DK, DV, NW>, (T*)out, (const T*)q,
                               (const T*)k_pool, (const T*)v_pool, req_to_token, req_pool_indices, seq_lens, H, G,
                               q_stride, out_stride, r2t_stride, sm_scale, window, sinks, slopes, qtemp_coef,
-                              qtemp_every, softcap, Gv, v_slot));
+                              qtemp_every, softcap, Gv, v_slot, kb));
   return 0;
 }
 
@@ -570,31 +582,31 @@ int attn_general_mma_decode_try(void* out, const void* q, const void* k_pool, co
                                 const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
                                 int64_t batch, int H, int G, int dk, int dv, int64_t q_stride, int64_t out_stride,
                                 int64_t r2t_stride, float sm_scale, int window, const float* sinks, const float* slopes,
-                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, int dtype,
-                                cudaStream_t stream) {
+                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb,
+                                int dtype, cudaStream_t stream) {
   if (dtype != SPD_BF16 && dtype != SPD_F16) return 1;
   if (v_slot % 8 != 0) return 1;
   if ((int64_t)G * ((H / G + 15) / 16) > 65535 || batch >= (1ll << 31)) return 1;
   if (q_stride % 8 != 0 || !aligned16(q) || !aligned16(k_pool) || !aligned16(v_pool)) return 1;
   // short windows do not fill eight warps: four warps then leave room for more CTAs per SM
-  const bool wide = window <= 0 || window > 4 * kGdTK;
+  const bool wide = window <= 0 || window > 4 * kGdTK || kb.size > 0;
 #define SPD_GD_CASE(DKV, DVV)                                                                                         \
   if (dk == DKV && dv == DVV) {                                                                                       \
     if (dtype == SPD_BF16)                                                                                            \
       return wide ? gd_launch_nw<__nv_bfloat16, DKV, DVV, 8>(out, q, k_pool, v_pool, req_to_token, req_pool_indices,  \
                                                              seq_lens, batch, H, G, q_stride, out_stride, r2t_stride, \
                                                              sm_scale, window, sinks, slopes, qtemp_coef, qtemp_every, \
-                                                             softcap, Gv, v_slot, stream)                                                  \
+                                                             softcap, Gv, v_slot, kb, stream)                                                  \
                   : gd_launch_nw<__nv_bfloat16, DKV, DVV, 4>(out, q, k_pool, v_pool, req_to_token, req_pool_indices,  \
                                                              seq_lens, batch, H, G, q_stride, out_stride, r2t_stride, \
                                                              sm_scale, window, sinks, slopes, qtemp_coef, qtemp_every, \
-                                                             softcap, Gv, v_slot, stream);                                                 \
+                                                             softcap, Gv, v_slot, kb, stream);                                                 \
     return wide ? gd_launch_nw<__half, DKV, DVV, 8>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, \
                                                     batch, H, G, q_stride, out_stride, r2t_stride, sm_scale, window,  \
-                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, stream)                   \
+                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, stream)                   \
                 : gd_launch_nw<__half, DKV, DVV, 4>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, \
                                                     batch, H, G, q_stride, out_stride, r2t_stride, sm_scale, window,  \
-                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, stream);                  \
+                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, stream);                  \
   }
   SPD_GD_CASE(32, 32)
   SPD_GD_CASE(64, 64)

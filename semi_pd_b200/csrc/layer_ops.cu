@@ -1,7 +1,7 @@
 // Small operators around the mixers and feed-forwards of the hybrid families, each in 16- and 32-bit:
 // an embedding that adds a sinusoidal position vector, the cast that joins two fp32 streams into one
 // GEMM operand, plain (ungated) activations, an RMS norm that writes its rows into a cache pool, a
-// per-head sigmoid gate, and an in-place scale of fp32 logits.  They follow hybrid_ops.cu's
+// per-head sigmoid gate, and an in-place scale or soft cap of fp32 logits.  They follow hybrid_ops.cu's
 // conventions (C ABI, no allocation, no sync); the reference has no model that needs them.
 #include "common.cuh"
 #include "ptx.cuh"
@@ -199,6 +199,14 @@ scale_f32_kernel(float* __restrict__ x, int64_t n, float alpha) {
     x[i] *= alpha;
 }
 
+__global__ void __launch_bounds__(kLayThreads)
+softcap_f32_kernel(float* __restrict__ x, int64_t n, float cap) {
+  griddep_wait();
+  griddep_launch_dependents();
+  for (int64_t i = blockIdx.x * (int64_t)kLayThreads + threadIdx.x; i < n; i += (int64_t)gridDim.x * kLayThreads)
+    x[i] = cap * tanhf(x[i] / cap);
+}
+
 inline unsigned flat_grid(int64_t n) {
   const int64_t blocks = (n + kLayThreads - 1) / kLayThreads;
   return (unsigned)(blocks < 8192 ? (blocks > 0 ? blocks : 1) : 8192);
@@ -300,6 +308,14 @@ int spd_scale_f32(float* x, int64_t n, float alpha, spd_stream_t stream) {
   if (n <= 0) return 0;
   SPD_CUDA(launch(scale_f32_kernel, dim3(flat_grid(n)), dim3(kLayThreads), 0, as_stream(stream), pdl_enabled(), x, n,
                   alpha));
+  return 0;
+}
+
+int spd_softcap_f32(float* x, int64_t n, float cap, spd_stream_t stream) {
+  SPD_REQUIRE(x && cap > 0.f, SPD_E_BADARG, "spd_softcap_f32: null pointer or cap not positive");
+  if (n <= 0) return 0;
+  SPD_CUDA(launch(softcap_f32_kernel, dim3(flat_grid(n)), dim3(kLayThreads), 0, as_stream(stream), pdl_enabled(), x, n,
+                  cap));
   return 0;
 }
 

@@ -4,7 +4,9 @@
 //     block adds in front of its first layer),
 //   * rotary positions over strided "segments" (q, k, v of a merged projection, or the rotated slice of a
 //     latent attention's queries and keys), in the paired or the half-split layout, with the biases of the
-//     projections added first and the cache write fused,
+//     projections added first, an RMS norm per head (with or without a weight) where a segment asks for one,
+//     and the cache write fused,
+//   * the fp32 residual update of layers that norm a sublayer's OUTPUT,
 //   * the step between an attention and its output projection: an elementwise sigmoid gate, optionally on
 //     the unit-RMS difference of two attention maps.
 // Everything is computed in fp32; 16-bit only at the loads and stores.
@@ -108,6 +110,9 @@ struct RotarySegment {
   void* dst;          // head h of token t goes to dst + (to_pool ? loc[t] : t) * dst_row + h * dst_head
   int64_t src_row, dst_row;
   int32_t heads, head_dim, rot, src_head, dst_head, to_pool;
+  const float* norm_w;  // [head_dim] or null (plain unit RMS); read when norm != 0
+  int32_t norm;         // RMS norm over the head's channels, after the bias and before the rotation
+  float norm_eps;
 };
 struct RotarySegments {
   RotarySegment seg[4];
@@ -217,6 +222,201 @@ rotary_segments_vec_kernel(RotarySegments segs, const int64_t* __restrict__ posi
   }
 }
 
+// The form with per-head norms: a warp per (token, head), the head's channels in shared memory between the norm and
+// the rotation.  VEC consecutive channels per lane and step (head_dim a multiple of 32 VEC for every segment, rows and
+// heads aligned to VEC elements), else VEC = 1.
+constexpr int kRotNormMaxDim = 512;
+template <typename T, int VEC>
+struct alignas(sizeof(T) * VEC) RotVec {
+  T e[VEC];
+};
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128)
+rotary_segments_norm_kernel(RotarySegments segs, const int64_t* __restrict__ positions, const int64_t* __restrict__ loc,
+                            const float* __restrict__ cos_sin, int rot_max, int64_t max_positions, int paired,
+                            int dim_max) {
+  griddep_wait();
+  griddep_launch_dependents();
+  extern __shared__ __align__(16) float rn_smem[];  // [4][dim_max]
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float* xs = rn_smem + warp * dim_max;
+  const int64_t t = blockIdx.x;
+  int64_t p = positions[t];
+  p = p < 0 ? 0 : (p < max_positions ? p : max_positions - 1);
+  const float* cs = cos_sin != nullptr ? cos_sin + p * rot_max : nullptr;
+  const int half_max = rot_max >> 1;
+  const int64_t slot = loc != nullptr ? loc[t] : 0;
+  int h0 = 0;  // heads of the segments before this one: head number n of the token goes to warp n mod 4
+  for (int sidx = 0; sidx < segs.n; ++sidx) {
+    const RotarySegment& sg = segs.seg[sidx];
+    const T* src = reinterpret_cast<const T*>(sg.src) + t * sg.src_row;
+    T* dst = reinterpret_cast<T*>(sg.dst) + (sg.to_pool ? slot : t) * sg.dst_row;
+    const int half = sg.rot >> 1, dim = sg.head_dim;
+    for (int h = (warp - h0) & 3; h < sg.heads; h += 4) {
+      const T* sp = src + h * sg.src_head;
+      const float* bs = sg.bias != nullptr ? sg.bias + h * dim : nullptr;
+      float ss = 0.f;
+      for (int d0 = lane * VEC; d0 < dim; d0 += 32 * VEC) {
+        const RotVec<T, VEC> v = *reinterpret_cast<const RotVec<T, VEC>*>(sp + d0);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const float x = to_f32<T>(v.e[e]) + (bs != nullptr ? bs[d0 + e] : 0.f);
+          ss = fmaf(x, x, ss);
+          xs[d0 + e] = x;
+        }
+      }
+      float inv = 1.f;
+      if (sg.norm) inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + sg.norm_eps);
+      const float* nw = sg.norm ? sg.norm_w : nullptr;
+      __syncwarp();
+      for (int d0 = lane * VEC; d0 < dim; d0 += 32 * VEC) {
+        RotVec<T, VEC> o;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const int d = d0 + e;
+          float y = xs[d] * inv * (nw != nullptr ? nw[d] : 1.f);
+          if (d < sg.rot) {
+            int pd, i;
+            bool first;
+            if (paired) { pd = d ^ 1; i = d >> 1; first = (d & 1) == 0; }
+            else { first = d < half; pd = first ? d + half : d - half; i = first ? d : d - half; }
+            const float yp = xs[pd] * inv * (nw != nullptr ? nw[pd] : 1.f);
+            const float c = cs[i], sn = cs[half_max + i];
+            y = first ? y * c - yp * sn : y * c + yp * sn;
+          }
+          o.e[e] = from_f32<T>(y);
+        }
+        *reinterpret_cast<RotVec<T, VEC>*>(dst + h * sg.dst_head + d0) = o;
+      }
+      __syncwarp();  // the next head overwrites xs
+    }
+    h0 += sg.heads;
+  }
+}
+
+// The residual update of a layer that norms its sublayer's output: x[row] += y / rms(y) * coef (y null: no update),
+// then out = x in T, or (w given) x / rms(x) * (off + w).  One CTA per row; a row of up to NV vectors per thread stays
+// in registers (VEC = 1: any size, read twice).
+constexpr int kPostThreads = 256;
+__device__ __forceinline__ float post_block_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int i = 0; i < kPostThreads / 32; ++i) t += red[i];
+  __syncthreads();
+  return t;
+}
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(kPostThreads)
+residual_postnorm_vec_kernel(T* __restrict__ out, float* __restrict__ x, const T* __restrict__ y,
+                             const float* __restrict__ coef, const T* __restrict__ w, int64_t dim, float eps, float off) {
+  griddep_wait();
+  griddep_launch_dependents();
+  constexpr int N = Vec16<T>::kN;
+  __shared__ float red[kPostThreads / 32];
+  const int64_t row = blockIdx.x;
+  float xv[NV][N], yv[NV][N];
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int64_t i = ((int64_t)v * kPostThreads + threadIdx.x) * N;
+    if (i < dim) {
+#pragma unroll
+      for (int e = 0; e < N; e += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(x + row * dim + i + e);
+        xv[v][e] = f.x; xv[v][e + 1] = f.y; xv[v][e + 2] = f.z; xv[v][e + 3] = f.w;
+      }
+      if (y != nullptr) {
+        const Vec16<T> a = ldv(y + row * dim + i);
+#pragma unroll
+        for (int e = 0; e < N; ++e) {
+          yv[v][e] = to_f32<T>(a.e()[e]);
+          ss = fmaf(yv[v][e], yv[v][e], ss);
+        }
+      }
+    }
+  }
+  if (y != nullptr) {
+    const float inv = 1.0f / sqrtf(post_block_sum(ss, red) / (float)dim + eps);
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int64_t i = ((int64_t)v * kPostThreads + threadIdx.x) * N;
+      if (i < dim) {
+#pragma unroll
+        for (int e = 0; e < N; e += 4) {
+          const float4 c = *reinterpret_cast<const float4*>(coef + i + e);
+          xv[v][e] += yv[v][e] * inv * c.x;
+          xv[v][e + 1] += yv[v][e + 1] * inv * c.y;
+          xv[v][e + 2] += yv[v][e + 2] * inv * c.z;
+          xv[v][e + 3] += yv[v][e + 3] * inv * c.w;
+          *reinterpret_cast<float4*>(x + row * dim + i + e) =
+              make_float4(xv[v][e], xv[v][e + 1], xv[v][e + 2], xv[v][e + 3]);
+        }
+      }
+    }
+  }
+  if (out == nullptr) return;
+  float inv = 1.f;
+  if (w != nullptr) {
+    ss = 0.f;
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
+      if (((int64_t)v * kPostThreads + threadIdx.x) * N < dim) {
+#pragma unroll
+        for (int e = 0; e < N; ++e) ss = fmaf(xv[v][e], xv[v][e], ss);
+      }
+    inv = 1.0f / sqrtf(post_block_sum(ss, red) / (float)dim + eps);
+  }
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int64_t i = ((int64_t)v * kPostThreads + threadIdx.x) * N;
+    if (i < dim) {
+      Vec16<T> o, wv;
+      if (w != nullptr) wv = ldv(w + i);
+#pragma unroll
+      for (int e = 0; e < N; ++e)
+        o.e()[e] = from_f32<T>(w != nullptr ? xv[v][e] * inv * (off + to_f32<T>(wv.e()[e])) : xv[v][e]);
+      stv(out + row * dim + i, o);
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kPostThreads)
+residual_postnorm_kernel(T* __restrict__ out, float* __restrict__ x, const T* __restrict__ y,
+                         const float* __restrict__ coef, const T* __restrict__ w, int64_t dim, float eps, float off) {
+  griddep_wait();
+  griddep_launch_dependents();
+  __shared__ float red[kPostThreads / 32];
+  const int64_t row = blockIdx.x;
+  float* xr = x + row * dim;
+  float inv = 0.f, ss = 0.f;
+  if (y != nullptr) {
+    for (int64_t i = threadIdx.x; i < dim; i += kPostThreads) {
+      const float a = to_f32<T>(y[row * dim + i]);
+      ss = fmaf(a, a, ss);
+    }
+    inv = 1.0f / sqrtf(post_block_sum(ss, red) / (float)dim + eps);
+  }
+  ss = 0.f;
+  for (int64_t i = threadIdx.x; i < dim; i += kPostThreads) {
+    float v = xr[i];
+    if (y != nullptr) {
+      v += to_f32<T>(y[row * dim + i]) * inv * coef[i];
+      xr[i] = v;
+    }
+    if (out != nullptr && w == nullptr) out[row * dim + i] = from_f32<T>(v);
+    ss = fmaf(v, v, ss);
+  }
+  if (out == nullptr || w == nullptr) return;
+  inv = 1.0f / sqrtf(post_block_sum(ss, red) / (float)dim + eps);
+  for (int64_t i = threadIdx.x; i < dim; i += kPostThreads)  // a thread reads back the elements it wrote
+    out[row * dim + i] = from_f32<T>(xr[i] * inv * (off + to_f32<T>(w[i])));
+}
+
 // out[t, h, c] = y[c] * sigmoid(gate[t, h * vdim + c]) with y = a[t, h, :] or, a2 given,
 // y = unit_rms(a - lambda a2) * post  (unit RMS over the head's vdim values, eps inside the root).
 template <typename T>
@@ -300,6 +500,29 @@ int spd_residual_tanh_norm(void* out, float* x, const void* a, const float* x0, 
   return 0;
 }
 
+int spd_residual_postnorm(void* out, float* x, const void* y, const float* coef, const void* w, int64_t rows, int64_t dim,
+                          float eps, float weight_offset, int dtype, spd_stream_t stream) {
+  SPD_REQUIRE(x && (y == nullptr) == (coef == nullptr) && (out != nullptr || w == nullptr) && (out || y), SPD_E_BADARG,
+              "spd_residual_postnorm: null pointer");
+  SPD_REQUIRE(rows >= 0 && dim > 0, SPD_E_BADARG, "spd_residual_postnorm: bad sizes");
+  if (rows == 0) return 0;
+  SPD_DISPATCH_ANY(dtype, {
+    constexpr int N = 16 / (int)sizeof(T);
+    const int64_t nv = (dim / N + kPostThreads - 1) / kPostThreads;
+    if (dim % N == 0 && nv <= 4 && aligned16(out) && aligned16(x) && aligned16(y) && aligned16(coef) && aligned16(w)) {
+      auto kern = nv == 1   ? residual_postnorm_vec_kernel<T, 1>
+                  : nv == 2 ? residual_postnorm_vec_kernel<T, 2>
+                            : residual_postnorm_vec_kernel<T, 4>;
+      SPD_CUDA(launch(kern, dim3((unsigned)rows), dim3(kPostThreads), 0, as_stream(stream), pdl_enabled(), (T*)out, x,
+                      (const T*)y, coef, (const T*)w, dim, eps, weight_offset));
+    } else {
+      SPD_CUDA(launch(residual_postnorm_kernel<T>, dim3((unsigned)rows), dim3(kPostThreads), 0, as_stream(stream),
+                      pdl_enabled(), (T*)out, x, (const T*)y, coef, (const T*)w, dim, eps, weight_offset));
+    }
+  });
+  return 0;
+}
+
 int spd_rotary_segments(const spd_rotary_segment_t* segments, int num_segments, const int64_t* positions,
                         const int64_t* loc, const float* cos_sin, int rot_max, int64_t max_positions, int paired,
                         int64_t tokens, int dtype, spd_stream_t stream) {
@@ -314,9 +537,35 @@ int spd_rotary_segments(const spd_rotary_segment_t* segments, int num_segments, 
     SPD_REQUIRE(s.rot == 0 || cos_sin != nullptr, SPD_E_BADARG, "spd_rotary_segments: rotation without a table");
     SPD_REQUIRE(!s.to_pool || loc != nullptr, SPD_E_BADARG, "spd_rotary_segments: a cache segment needs slot ids");
     segs.seg[i] = RotarySegment{s.src, s.bias, s.dst, s.src_row, s.dst_row, s.heads, s.head_dim, s.rot, s.src_head,
-                                s.dst_head, s.to_pool};
+                                s.dst_head, s.to_pool, s.norm_w, s.norm, s.norm_eps};
   }
   if (tokens == 0) return 0;
+  int dim_max = 0, step = 4;  // form with norms: the widest step every segment's sizes allow
+  bool any_norm = false;
+  for (int i = 0; i < num_segments; ++i) {
+    const RotarySegment& s = segs.seg[i];
+    any_norm = any_norm || s.norm != 0;
+    dim_max = s.head_dim > dim_max ? s.head_dim : dim_max;
+    const int64_t align = dtype == SPD_F32 ? 4 : 2;
+    while (step > 1 && (s.head_dim % (32 * step) != 0 || s.src_head % step != 0 || s.dst_head % step != 0 ||
+                        s.src_row % step != 0 || s.dst_row % step != 0 ||
+                        reinterpret_cast<uintptr_t>(s.src) % (step * align) != 0 ||
+                        reinterpret_cast<uintptr_t>(s.dst) % (step * align) != 0))
+      step >>= 1;
+  }
+  if (any_norm) {
+    SPD_REQUIRE(dim_max <= kRotNormMaxDim, SPD_E_SHAPE, "spd_rotary_segments: normed heads of %d channels (max %d)",
+                dim_max, kRotNormMaxDim);
+    const int pad = (dim_max + 3) / 4 * 4;
+    SPD_DISPATCH_ANY(dtype, {
+      auto kern = step == 4   ? rotary_segments_norm_kernel<T, 4>
+                  : step == 2 ? rotary_segments_norm_kernel<T, 2>
+                              : rotary_segments_norm_kernel<T, 1>;
+      SPD_CUDA(launch(kern, dim3((unsigned)tokens), dim3(128), sizeof(float) * 4 * (size_t)pad, as_stream(stream),
+                      pdl_enabled(), segs, positions, loc, cos_sin, rot_max, max_positions, paired, pad));
+    });
+    return 0;
+  }
   const int vecn = dtype == SPD_F32 ? 4 : 8;
   bool vec = true;
   for (int i = 0; i < num_segments; ++i) {

@@ -387,7 +387,7 @@ class RecurrentStatePool:
     0 ignores what the slot held before (no clearing on reuse).  `layer_shapes[l]` is (heads,
     head_dim, v_dim) or None for layers without state.  `shift_dims[l]` (optional) is the row size of
     a second, vector-valued state of layer l — the previous token's mixer input of a token-shift
-    mixer, `shift[l]` fp32 [slots, dim] — or None.  `token_state`: the pool also keeps every request's last
+    mixer, the last inputs of a short convolution, `shift[l]` fp32 [slots, dim] — or None.  `token_state`: the pool also keeps every request's last
     token id (`prev_token` int32 [slots]) for an embedding that looks at pairs of tokens."""
 
     def __init__(self, num_slots: int, layer_shapes: Sequence[Optional[Tuple[int, int, int]]], device: str,
@@ -426,11 +426,20 @@ class HybridTokenToKVPool(KVCache):
     keys: several attention maps over one set of values); layers with None (recurrent mixers) own nothing here.  All
     layers share the slot ids of one TokenToKVPoolAllocator, as in MHATokenToKVPool.  `dtype` may be
     float32.  The recurrent layers' state pool travels with this object (`state_pool`), so both
-    workers of a GPU see it through the one pool they already share."""
+    workers of a GPU see it through the one pool they already share.
+
+    `kv_from[l]` = j: layer l reads layer j's buffers instead of owning any (its own shape is None).
+
+    `block_sizes[l]` = P: layer l also sees pooled blocks of P tokens (one mean key and value each).  Their rows lie
+    behind the token rows of the buffers they are read from — per block size that any layer over those buffers uses, one
+    region of ceil(run_len / P) rows for every run of the allocator, a block belonging to the run its last token is in.
+    A block row is therefore taken, reused and freed with the run of slots it summarises (csrc/key_blocks.cuh has the
+    same address rule); `get_blocks(l)` is (P, run_len, first row of the region)."""
 
     def __init__(self, size: int, page_size: int, dtype: torch.dtype,
                  layer_shapes: Sequence[Optional[Tuple[int, int, int]]], device: str,
-                 state_pool: Optional[RecurrentStatePool] = None):
+                 state_pool: Optional[RecurrentStatePool] = None, kv_from: Optional[Sequence[Optional[int]]] = None,
+                 block_sizes: Optional[Sequence[Optional[int]]] = None, run_len: int = DEFAULT_RUN_LEN):
         if page_size != 1:
             raise NotImplementedError("semi-PD path is token-granular: page_size must be 1")
         self.size = size
@@ -441,24 +450,59 @@ class HybridTokenToKVPool(KVCache):
         self.layer_shapes = list(layer_shapes)
         self.layer_num = len(self.layer_shapes)
         self.state_pool = state_pool
-        rows = size + page_size
+        self.run_len = int(run_len)
+        self.owner = self._owners(self.layer_shapes, kv_from)
+        runs = -(-size // self.run_len)
+        rows = [size + page_size] * self.layer_num   # rows of an owner's buffers
+        regions: Dict[Tuple[int, int], int] = {}     # (owner, block size) -> first row
+        self._blocks: List[Optional[Tuple[int, int, int]]] = [None] * self.layer_num
+        self._writes_blocks = [False] * self.layer_num
+        for i, p in enumerate(block_sizes or []):
+            if p:
+                key = (self.owner[i], int(p))
+                if key not in regions:
+                    regions[key] = rows[key[0]]
+                    rows[key[0]] += runs * -(-self.run_len // key[1])
+                    self._writes_blocks[i] = True  # layers run in order: this is the first that reads the region
+                self._blocks[i] = (key[1], self.run_len, regions[key])
         self.k_buffer: List[Optional[torch.Tensor]] = []
         self.v_buffer: List[Optional[torch.Tensor]] = []
-        for s in self.layer_shapes:
-            self.k_buffer.append(torch.zeros((rows, s[0], s[1]), dtype=dtype, device=device) if s else None)
+        for i, s in enumerate(self.layer_shapes):
+            self.k_buffer.append(torch.zeros((rows[i], s[0], s[1]), dtype=dtype, device=device) if s else None)
             self.v_buffer.append(None if not s else self.k_buffer[-1] if s[2] == 0 else
-                                 torch.zeros((rows, s[3] if len(s) > 3 else s[0], s[2]), dtype=dtype, device=device))
+                                 torch.zeros((rows[i], s[3] if len(s) > 3 else s[0], s[2]), dtype=dtype, device=device))
+        for i, j in enumerate(self.owner):
+            self.k_buffer[i], self.v_buffer[i] = self.k_buffer[j], self.v_buffer[j]
 
     @staticmethod
-    def bytes_per_token(layer_shapes, dtype: torch.dtype) -> int:
+    def _owners(layer_shapes, kv_from) -> List[int]:
+        owner = [i if j is None else int(j) for i, j in enumerate(kv_from or [None] * len(layer_shapes))]
+        for i, j in enumerate(owner):
+            if j != i and (not 0 <= j < i or owner[j] != j or layer_shapes[j] is None or layer_shapes[i] is not None):
+                raise ValueError(f"layer {i}: kv_from {j} must name an earlier layer with keys and values of its own")
+        return owner
+
+    @classmethod
+    def bytes_per_token(cls, layer_shapes, dtype: torch.dtype, kv_from=None, block_sizes=None,
+                        run_len: int = DEFAULT_RUN_LEN) -> int:
+        """Bytes a token takes in all layers, its share of the block rows included (rounded up)."""
         esz = torch.empty((), dtype=dtype).element_size()
-        return sum((s[0] * s[1] + (s[3] if len(s) > 3 else s[0]) * s[2]) * esz for s in layer_shapes if s is not None)
+        row = [(s[0] * s[1] + (s[3] if len(s) > 3 else s[0]) * s[2]) * esz if s is not None else 0 for s in layer_shapes]
+        owner = cls._owners(layer_shapes, kv_from)
+        pooled = sum(row[o] * -(-run_len // p) for o, p in {(owner[i], int(p)) for i, p in enumerate(block_sizes or []) if p})
+        return sum(row) + -(-pooled // run_len)
 
     def get_kv_size_bytes(self):
-        k = sum(b.numel() * b.element_size() for b in self.k_buffer if b is not None)
-        v = sum(b.numel() * b.element_size() for b, kb in zip(self.v_buffer, self.k_buffer)
-                if b is not None and b is not kb)
-        return k, v
+        own = [(self.k_buffer[i], self.v_buffer[i]) for i in range(self.layer_num)
+               if self.owner[i] == i and self.k_buffer[i] is not None]
+        return (sum(k.numel() * k.element_size() for k, _ in own),
+                sum(v.numel() * v.element_size() for k, v in own if v is not k))
+
+    def get_blocks(self, layer_id: int) -> Optional[Tuple[int, int, int]]:
+        return self._blocks[layer_id]
+
+    def writes_blocks(self, layer_id: int) -> bool:
+        return self._writes_blocks[layer_id]
 
     def get_key_buffer(self, layer_id: int):
         return self.k_buffer[layer_id]

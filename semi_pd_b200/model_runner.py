@@ -120,8 +120,10 @@ class ModelRunner:
         cfg = self.model_config
         esz = torch.tensor([], dtype=self.kv_cache_dtype).element_size()
         if getattr(cfg, "layer_specs", None) is not None:
-            kv_shapes = self.model.cache_shapes()[0]
-            cell = max(HybridTokenToKVPool.bytes_per_token(kv_shapes, self.kv_cache_dtype), 64)
+            kv_shapes, _, *more = self.model.cache_shapes()
+            extras = more[1] if len(more) > 1 else {}
+            cell = max(HybridTokenToKVPool.bytes_per_token(kv_shapes, self.kv_cache_dtype, extras.get("kv_from"),
+                                                           extras.get("block_sizes")), 64)
         elif getattr(cfg, "model_type", "llama") == "deepseek_v2":
             cell = (cfg.kv_lora_rank + cfg.qk_rope_head_dim) * cfg.num_hidden_layers * esz  # model_runner.py:930-936
         else:
@@ -151,12 +153,13 @@ class ModelRunner:
         self.req_to_token_pool = ReqToTokenPool(size=max_num_reqs + 1, max_context_len=ctx + 4,
                                                 device=self.device)
         if hybrid:
-            # (kv shapes, matrix-state shapes[, vector-state sizes[, {"token_state": bool}]]) per layer
+            # (kv shapes, matrix-state shapes[, vector-state sizes[, {"token_state": bool, "kv_from": [layer | None],
+            # "block_sizes": [tokens per pooled block | None]}]]) per layer
             kv_shapes, state_shapes, *more = self.model.cache_shapes()
             extras = more[1] if len(more) > 1 else {}
             self.token_to_kv_pool = HybridTokenToKVPool(
                 self.max_total_num_tokens, page_size=1, dtype=self.kv_cache_dtype, layer_shapes=kv_shapes,
-                device=self.device,
+                device=self.device, kv_from=extras.get("kv_from"), block_sizes=extras.get("block_sizes"),
                 state_pool=RecurrentStatePool(max_num_reqs + 1, state_shapes, device=self.device,
                                               shift_dims=more[0] if more else None,
                                               token_state=bool(extras.get("token_state"))))

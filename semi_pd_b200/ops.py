@@ -912,13 +912,14 @@ def attn_general(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, re
                  sinks: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None, qtemp_coef: float = 0.0,
                  qtemp_every: int = 0, seq_lens=None, prefix_lens=None, extend_lens=None, extend_start_loc=None,
                  max_extend_len: int = 0, softcap: float = 0.0, num_v_heads: int = 0,
-                 v_slot_stride: int = 0) -> torch.Tensor:
+                 v_slot_stride: int = 0, blocks: Optional[tuple] = None) -> torch.Tensor:
     """Windowed / sink / distance-biased softmax attention over the paged pool; decode (seq_lens) or
     ragged extend (prefix_lens, extend_lens, extend_start_loc).  q [T, H·head_dim] → [T, H·v_dim].
     max_extend_len > 0 (a host-side bound of extend_lens) lets 16-bit prefill run on the tensor cores.
     softcap > 0 caps the scaled scores by softcap · tanh(· / softcap); num_v_heads < num_kv_heads: key head g
     reads value head g mod num_v_heads; v_slot_stride: elements between two slots of v_pool (values that are
-    the first v_dim columns of wider rows)."""
+    the first v_dim columns of wider rows).  blocks (size, run_len, base): besides its window a query sees one pooled key
+    and value per block of `size` tokens that lies wholly before the window (rows written by pool_key_blocks)."""
     _cuda(q, k_pool, v_pool, req_to_token, req_pool_indices, sinks, slopes)
     T = q.shape[0]
     if q.dim() != 2 or q.stride(1) != 1:
@@ -932,14 +933,37 @@ def attn_general(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, re
         if t is not None and t.dtype != torch.float32:
             raise RuntimeError("attn_general: sinks and slopes are fp32")
     out = torch.empty((T, num_q_heads * v_dim), device=q.device, dtype=q.dtype)
-    check(lib.spd_attn_general_ex(out.data_ptr(), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
+    size, run_len, base = blocks or (0, 0, 0)
+    check(lib.spd_attn_general_blocks(out.data_ptr(), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
                                   req_to_token.data_ptr(), req_pool_indices.data_ptr(), _ptr(seq_lens), _ptr(prefix_lens),
                                   _ptr(extend_lens), _ptr(extend_start_loc), req_pool_indices.numel(), T, num_q_heads,
                                   num_kv_heads, head_dim, v_dim, q.stride(0), out.stride(0), req_to_token.stride(0),
                                   float(sm_scale), int(window), _ptr(sinks), _ptr(slopes), float(qtemp_coef),
                                   int(qtemp_every), int(max_extend_len), float(softcap or 0.0), int(num_v_heads),
-                                  int(v_slot_stride), _dta(q), _stream()), "spd_attn_general")
+                                  int(v_slot_stride), int(size), int(run_len), int(base), _dta(q), _stream()),
+          "spd_attn_general")
     return out
+
+
+def pool_key_blocks(k_pool: torch.Tensor, v_pool: Optional[torch.Tensor], req_to_token, req_pool_indices, blocks: tuple,
+                    seq_lens=None, prefix_lens=None, extend_lens=None, max_extend_len: int = 0) -> None:
+    """Writes the rows of the blocks that a batch's new tokens complete: the mean of each block's cached keys and values
+    (summed in fp32).  k_pool / v_pool [rows, ...] contiguous, the new tokens' rows already in them; blocks (size,
+    run_len, base) as attn_general.  Decode (seq_lens) or ragged extend (max_extend_len: bound of extend_lens)."""
+    _cuda(k_pool, v_pool, req_to_token, req_pool_indices)
+    if not k_pool.is_contiguous() or (v_pool is not None and (not v_pool.is_contiguous() or v_pool.dtype != k_pool.dtype)):
+        raise RuntimeError("pool_key_blocks: the pools are contiguous and share a dtype")
+    if req_pool_indices.dtype != torch.int64 or (seq_lens is not None and seq_lens.dtype != torch.int64):
+        raise RuntimeError("pool_key_blocks: req_pool_indices and seq_lens must be int64")
+    for t in (prefix_lens, extend_lens):
+        if t is not None and t.dtype != torch.int32:
+            raise RuntimeError("pool_key_blocks: prefix_lens / extend_lens must be int32")
+    size, run_len, base = blocks
+    check(lib.spd_pool_key_blocks(k_pool.data_ptr(), _ptr(v_pool), req_to_token.data_ptr(), req_pool_indices.data_ptr(),
+                                  _ptr(seq_lens), _ptr(prefix_lens), _ptr(extend_lens), req_pool_indices.numel(),
+                                  int(max_extend_len), req_to_token.stride(0), k_pool[0].numel(),
+                                  v_pool[0].numel() if v_pool is not None else 0, int(size), int(run_len), int(base),
+                                  _dta(k_pool), _stream()), "spd_pool_key_blocks")
 
 
 def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, req_pool_indices,
@@ -1133,24 +1157,30 @@ def residual_tanh_norm(x: torch.Tensor, weight: Optional[torch.Tensor], bias: Op
 
 def rotary_segment(src: torch.Tensor, dst: torch.Tensor, heads: int, head_dim: int, rot: int = 0,
                    bias: Optional[torch.Tensor] = None, src_head: Optional[int] = None, dst_head: Optional[int] = None,
-                   to_pool: bool = False) -> _lib.RotarySegment:
+                   to_pool: bool = False, norm_eps: Optional[float] = None,
+                   norm_weight: Optional[torch.Tensor] = None) -> _lib.RotarySegment:
     """One piece of rotary_segments: src / dst are 2-D views whose first element is the first head's first channel
-    (row stride = stride(0); src_head / dst_head default to head_dim)."""
-    _cuda(src, dst, bias)
+    (row stride = stride(0); src_head / dst_head default to head_dim).  norm_eps (not None): every head is brought to
+    unit RMS over its channels after the bias and before the rotation, times norm_weight (fp32 [head_dim], optional)."""
+    _cuda(src, dst, bias, norm_weight)
+    if norm_weight is not None and (norm_eps is None or norm_weight.dtype != torch.float32
+                                    or not norm_weight.is_contiguous() or norm_weight.numel() != head_dim):
+        raise RuntimeError("rotary_segment: norm_weight is contiguous fp32 [head_dim], with norm_eps")
     if src.stride(-1) != 1 or dst.stride(-1) != 1 or src.dtype != dst.dtype:
         raise RuntimeError("rotary_segment: src and dst have contiguous rows and one dtype")
     if bias is not None and (bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() != heads * head_dim):
         raise RuntimeError("rotary_segment: bias is contiguous fp32 [heads * head_dim]")
     seg = _lib.RotarySegment(src.data_ptr(), _ptr(bias), dst.data_ptr(), src.stride(0), dst.stride(0), heads, head_dim, rot,
                              head_dim if src_head is None else src_head, head_dim if dst_head is None else dst_head,
-                             1 if to_pool else 0)
-    seg.keep = (src, dst, bias)  # the descriptor holds raw pointers: the tensors live as long as it does
+                             1 if to_pool else 0, _ptr(norm_weight), 0 if norm_eps is None else 1,
+                             0.0 if norm_eps is None else float(norm_eps))
+    seg.keep = (src, dst, bias, norm_weight)  # the descriptor holds raw pointers: the tensors live as long as it does
     return seg
 
 
 def rotary_segments(segments, positions: torch.Tensor, cos_sin: Optional[torch.Tensor], dtype: torch.dtype,
                     loc: Optional[torch.Tensor] = None, paired: bool = False) -> None:
-    """Bias + partial rotation + scatter of up to four strided segments in one launch (see rotary_segment).
+    """Bias [+ norm per head] + partial rotation + scatter of up to four strided segments in one launch (rotary_segment).
     cos_sin fp32 [positions, rot_max] = cos ‖ sin; paired: channel 2 i turns with 2 i + 1, else i with i + rot / 2."""
     _cuda(positions, cos_sin, loc)
     if positions.dtype != torch.int64 or (loc is not None and loc.dtype != torch.int64):
@@ -1178,6 +1208,106 @@ def heads_gate(a: torch.Tensor, gate: torch.Tensor, heads: int, vdim: int, a2: O
     check(lib.spd_heads_gate(out.data_ptr(), a.data_ptr(), _ptr(a2), gate.data_ptr(), T, heads, vdim, a.stride(0),
                              gate.stride(0), out.stride(0), float(lam), float(eps), float(post), _dta(a), _stream()),
           "spd_heads_gate")
+    return out
+
+
+# ------------------------------------------------------------------------------------------------
+# norms on a sublayer's output, recurrences with one decay per head, short convolutions
+# ------------------------------------------------------------------------------------------------
+def residual_postnorm(x: torch.Tensor, y: Optional[torch.Tensor], coef: Optional[torch.Tensor], eps: float,
+                      dtype: torch.dtype, weight: Optional[torch.Tensor] = None, weight_offset: float = 0.0) -> torch.Tensor:
+    """x (fp32, in place) += y / rms(y) · coef (coef fp32 [dim]; y None: no update); → x in `dtype`, or with weight
+    x / rms(x) · (weight_offset + weight)."""
+    _cuda(x, y, coef, weight)
+    if x.dtype != torch.float32 or not x.is_contiguous() or x.dim() != 2:
+        raise RuntimeError("residual_postnorm: the residual stream is contiguous fp32 [T, dim]")
+    d = x.shape[1]
+    if y is not None and (y.dtype != dtype or not y.is_contiguous() or y.shape != x.shape):
+        raise RuntimeError("residual_postnorm: y matches x, is contiguous and has the output's dtype")
+    if (y is None) != (coef is None) or (coef is not None and (coef.dtype != torch.float32 or not coef.is_contiguous()
+                                                               or coef.numel() != d)):
+        raise RuntimeError("residual_postnorm: coef is contiguous fp32 [dim], given with y")
+    if weight is not None and (weight.dtype != dtype or not weight.is_contiguous() or weight.numel() != d):
+        raise RuntimeError("residual_postnorm: weight is [dim] in the output's dtype")
+    out = torch.empty(x.shape, device=x.device, dtype=dtype)
+    check(lib.spd_residual_postnorm(out.data_ptr(), x.data_ptr(), _ptr(y), _ptr(coef), _ptr(weight), x.shape[0], d,
+                                    float(eps), float(weight_offset), _dta(out), _stream()), "spd_residual_postnorm")
+    return out
+
+
+def softcap_f32_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x = cap · tanh(x / cap) in place (contiguous fp32)."""
+    _cuda(x)
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise RuntimeError("softcap_f32_: x is contiguous fp32")
+    check(lib.spd_softcap_f32(x.data_ptr(), x.numel(), float(cap), _stream()), "spd_softcap_f32")
+    return x
+
+
+def head_decay_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, state: torch.Tensor,
+                          req_pool_indices, num_heads: int, num_k_heads: int, head_dim: int, v_dim: int, form: str,
+                          dt_bias: torch.Tensor, a_log: torch.Tensor, skip: Optional[torch.Tensor] = None,
+                          b: Optional[torch.Tensor] = None, q_scale: float = 1.0, unit_eps: float = 1e-6, seq_lens=None,
+                          out_cache_loc=None, prefix_lens=None, extend_lens=None, extend_start_loc=None) -> torch.Tensor:
+    """Matrix-state recurrence with one decay exp(-exp(a_log) softplus(z + dt_bias)) per head and token over the
+    per-request state (fp32 [slots, heads, v_dim, head_dim], updated in place).  form "ssd": S = w S + dt k vᵀ, o = Sᵀ q
+    + skip v; form "delta": unit-length k and q, S = w S, then S += k (sigmoid(b) (v − Sᵀ k))ᵀ, o = Sᵀ q.  q / k
+    [T, num_k_heads · head_dim], v [T, heads · v_dim], z / b [T, heads] (row-strided views) → o fp32 [T, heads · v_dim]."""
+    _cuda(q, k, v, z, state, req_pool_indices, dt_bias, a_log, skip, b)
+    T = q.shape[0]
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (num_heads, v_dim, head_dim):
+        raise RuntimeError("head_decay_recurrence: the state is contiguous fp32 [slots, heads, v_dim, head_dim]")
+    if any(t.stride(1) != 1 or t.dtype != q.dtype for t in (q, k, v)) or z.dtype != q.dtype \
+            or (b is not None and b.dtype != q.dtype):
+        raise RuntimeError("head_decay_recurrence: q / k / v / z / b need contiguous rows and one dtype")
+    for t in (dt_bias, a_log, skip):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != num_heads or not t.is_contiguous()):
+            raise RuntimeError("head_decay_recurrence: dt_bias, a_log and skip are fp32 [heads]")
+    o = torch.empty((T, num_heads * v_dim), device=q.device, dtype=torch.float32)
+    check(lib.spd_head_decay(o.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), z.data_ptr(), _ptr(b),
+                             state.data_ptr(), req_pool_indices.data_ptr(), _ptr(seq_lens), _ptr(out_cache_loc),
+                             _ptr(prefix_lens), _ptr(extend_lens), _ptr(extend_start_loc), req_pool_indices.numel(),
+                             num_heads, num_k_heads, head_dim, v_dim, q.stride(0), k.stride(0), v.stride(0), z.stride(0),
+                             b.stride(0) if b is not None else 0, dt_bias.data_ptr(), a_log.data_ptr(), _ptr(skip),
+                             {"ssd": 0, "delta": 1}[form], float(q_scale), float(unit_eps), _dta(q), _stream()),
+          "spd_head_decay")
+    return o
+
+
+def short_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor],
+               req_pool_indices, seq_lens=None, out_cache_loc=None, prefix_lens=None, extend_lens=None,
+               extend_start_loc=None, max_extend_len: int = 0) -> torch.Tensor:
+    """silu of a causal convolution per channel within each request: x [T, channels] (row-strided view allowed), weight
+    [taps, channels] (the current token's last), bias [channels] or None.  The taps − 1 inputs before a request's first
+    new row live in state[slot] (fp32 [slots, (taps − 1) · channels]; zeros at position 0), updated in place."""
+    _cuda(x, weight, bias, state, req_pool_indices)
+    T, channels = x.shape
+    taps = weight.shape[0]
+    if x.stride(1) != 1 or weight.shape[1] != channels or not weight.is_contiguous() or weight.dtype != x.dtype \
+            or (bias is not None and (bias.dtype != x.dtype or bias.numel() != channels or not bias.is_contiguous())):
+        raise RuntimeError("short_conv: x [T, channels] with contiguous rows; weight [taps, channels] and bias in its dtype")
+    if taps > 1 and (state is None or state.dtype != torch.float32 or not state.is_contiguous()
+                     or state[0].numel() != (taps - 1) * channels):
+        raise RuntimeError("short_conv: the state is contiguous fp32 [slots, (taps - 1) * channels]")
+    out = torch.empty((T, channels), device=x.device, dtype=x.dtype)
+    check(lib.spd_short_conv(out.data_ptr(), x.data_ptr(), weight.data_ptr(), _ptr(bias), _ptr(state),
+                             req_pool_indices.data_ptr(), _ptr(seq_lens), _ptr(out_cache_loc), _ptr(prefix_lens),
+                             _ptr(extend_lens), _ptr(extend_start_loc), req_pool_indices.numel(), T, int(max_extend_len),
+                             channels, taps, x.stride(0), _dta(x), _stream()), "spd_short_conv")
+    return out
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    """y fp32 [T, n] · silu(z), each of `groups` equal parts of a row brought to unit RMS by itself, · weight [n]; in
+    z's dtype (z may be a row-strided view)."""
+    _cuda(y, z, weight)
+    T, n = y.shape
+    if y.dtype != torch.float32 or not y.is_contiguous() or z.stride(1) != 1 or weight.dtype != z.dtype \
+            or weight.numel() != n or not weight.is_contiguous() or n % groups:
+        raise RuntimeError("gated_group_norm: y is contiguous fp32 [T, n], weight [n] in z's dtype, n a multiple of groups")
+    out = torch.empty((T, n), device=y.device, dtype=z.dtype)
+    check(lib.spd_gated_group_norm(out.data_ptr(), y.data_ptr(), z.data_ptr(), weight.data_ptr(), T, groups, n // groups,
+                                   z.stride(0), float(eps), _dta(z), _stream()), "spd_gated_group_norm")
     return out
 
 

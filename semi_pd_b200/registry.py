@@ -14,6 +14,7 @@ _MODELS: Dict[str, Tuple[str, str]] = {
     "nupovik": ("nupovik", "NupovikForCausalLM"),
     "matepel": ("matepel", "MatepelForCausalLM"),
     "sugelix": ("sugelix", "SugelixForCausalLM"),
+    "fudonex": ("fudonex", "FudonexForCausalLM"),
 }
 
 
