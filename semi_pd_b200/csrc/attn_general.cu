@@ -473,15 +473,21 @@ kv_store_kernel(const T* __restrict__ k, const T* __restrict__ v, T* __restrict_
 }
 
 // Block rows of the blocks that a batch completes: the mean over the block's cache rows of K and V, as the cache holds
-// them, in fp32.  One CTA per (request, block that its new tokens may complete).
+// them, in fp32.  One CTA per (request, block that its new tokens may complete); a row's vectors (K, then V) go to
+// neighbouring threads, and where they leave threads over, TL of them share a vector by tokens (their sums meet in
+// shared memory, in a fixed order).
+constexpr int kPoolThreads = 128;
+constexpr int kPoolSlots = 512;  // slot numbers staged at a time
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kPoolThreads)
 pool_key_blocks_kernel(T* __restrict__ k_pool, T* __restrict__ v_pool, const int32_t* __restrict__ req_to_token,
                        const int64_t* __restrict__ req_pool_indices, const int64_t* __restrict__ seq_lens,
                        const int32_t* __restrict__ prefix_lens, const int32_t* __restrict__ extend_lens,
-                       int64_t r2t_stride, int64_t k_row, int64_t v_row, KeyBlocks kb) {
+                       int64_t r2t_stride, int64_t k_row, int64_t v_row, int tl_lanes, KeyBlocks kb) {
   griddep_wait();
   griddep_launch_dependents();
+  __shared__ int slots[kPoolSlots];
+  __shared__ float part[kPoolThreads * VEC];
   const int r = blockIdx.y;
   const int64_t pos0 = seq_lens != nullptr ? seq_lens[r] - 1 : (int64_t)prefix_lens[r];
   const int64_t end = seq_lens != nullptr ? pos0 + 1 : pos0 + extend_lens[r];  // tokens cached by now
@@ -492,22 +498,47 @@ pool_key_blocks_kernel(T* __restrict__ k_pool, T* __restrict__ v_pool, const int
   if (page[kb.size - 1] <= 0) return;  // a padded row of a captured batch
   const int64_t row = key_block_row(kb, page[kb.size - 1]);
   const float inv = 1.0f / (float)kb.size;
-  auto mean = [&](T* pool, int64_t n) {
-    for (int64_t c = threadIdx.x * VEC; c < n; c += 128 * VEC) {
-      float acc[VEC];
+  const int per = kPoolThreads / tl_lanes;  // vectors in flight
+  const int tl = threadIdx.x / per, lv = threadIdx.x - tl * per;
+  const int64_t kv = k_row / VEC, nv = kv + (v_pool != nullptr ? v_row / VEC : 0);
+  for (int64_t v0 = 0; v0 < nv; v0 += per) {
+    const int64_t v = v0 + lv;
+    const bool on = tl < tl_lanes && v < nv;
+    T* pool = v < kv ? k_pool : v_pool;
+    const int64_t n = v < kv ? k_row : v_row, c = (v < kv ? v : v - kv) * VEC;
+    float acc[VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
-#pragma unroll 4
-      for (int i = 0; i < kb.size; ++i) {
-        const T* src = pool + (int64_t)page[i] * n + c;
-        if constexpr (VEC == 1) {
-          acc[0] += to_f32<T>(src[0]);
-        } else {
-          const Vec16<T> x = ldv(src);
+    for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+    for (int i0 = 0; i0 < kb.size; i0 += kPoolSlots) {
+      const int m = kb.size - i0 < kPoolSlots ? kb.size - i0 : kPoolSlots;
+      __syncthreads();
+      for (int i = threadIdx.x; i < m; i += kPoolThreads) slots[i] = page[i0 + i];
+      __syncthreads();
+      if (on) {
+#pragma unroll 8
+        for (int i = tl; i < m; i += tl_lanes) {
+          const T* src = pool + (int64_t)slots[i] * n + c;
+          if constexpr (VEC == 1) {
+            acc[0] += to_f32<T>(src[0]);
+          } else {
+            const Vec16<T> x = ldv(src);
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) acc[e] += to_f32<T>(x.e()[e]);
+            for (int e = 0; e < VEC; ++e) acc[e] += to_f32<T>(x.e()[e]);
+          }
         }
       }
+    }
+    if (tl_lanes > 1) {
+      __syncthreads();
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) part[threadIdx.x * VEC + e] = acc[e];
+      __syncthreads();
+      if (tl == 0)
+        for (int x = 1; x < tl_lanes; ++x)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) acc[e] += part[(x * per + lv) * VEC + e];
+    }
+    if (on && tl == 0) {
       T* dst = pool + row * n + c;
       if constexpr (VEC == 1) {
         dst[0] = from_f32<T>(acc[0] * inv);
@@ -518,9 +549,7 @@ pool_key_blocks_kernel(T* __restrict__ k_pool, T* __restrict__ v_pool, const int
         stv(dst, x);
       }
     }
-  };
-  mean(k_pool, k_row);
-  if (v_pool != nullptr) mean(v_pool, v_row);
+  }
 }
 
 int attn_general_mma_try(void* out, const void* q, const void* k_pool, const void* v_pool, const int32_t* req_to_token,
@@ -575,9 +604,12 @@ int spd_pool_key_blocks(void* k_pool, void* v_pool, const int32_t* req_to_token,
     constexpr int N = 16 / (int)sizeof(T);
     const bool vec = k_row_elems % N == 0 && v_row_elems % N == 0 && aligned16(k_pool) && aligned16(v_pool);
     auto kern = vec ? pool_key_blocks_kernel<T, N> : pool_key_blocks_kernel<T, 1>;
-    SPD_CUDA(launch(kern, grid, dim3(128), 0, as_stream(stream), pdl_enabled(), (T*)k_pool, (T*)v_pool, req_to_token,
-                    req_pool_indices, seq_lens, prefix_lens, extend_lens, req_to_token_stride, k_row_elems, v_row_elems,
-                    kb));
+    const int64_t vecs = (k_row_elems + (v_pool != nullptr ? v_row_elems : 0)) / (vec ? N : 1);
+    int tl = 1;  // token lanes per vector
+    while (tl < 8 && tl * 2 <= block_size && vecs * tl * 2 <= kPoolThreads) tl *= 2;
+    SPD_CUDA(launch(kern, grid, dim3(kPoolThreads), 0, as_stream(stream), pdl_enabled(), (T*)k_pool, (T*)v_pool,
+                    req_to_token, req_pool_indices, seq_lens, prefix_lens, extend_lens, req_to_token_stride, k_row_elems,
+                    v_row_elems, tl, kb));
   });
   return 0;
 }

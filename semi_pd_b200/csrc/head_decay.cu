@@ -8,11 +8,15 @@
 //
 // Decode and ragged extend (chunked prefill, mixed batches) are one kernel: a CTA owns (request, head, 32 value
 // columns).  Eight lanes share a column pair, each with every eighth group of four state rows of the two columns in
-// registers (as packed fp32 pairs), so both products with the old state are three shuffles away from complete and a
-// token needs no block-wide barrier.  The delta rule reads the state once per token:
-//   S'^T k = w (S_(t-1)^T k),   o_t = w (S_(t-1)^T q) + (k . q) u_t
-// Separate producer warps prepare the next block of tokens in shared memory (loads, unit length, k . q, step size,
-// decay) while the consumer warps walk the current one; one block-wide barrier per token block.  The state is stored
+// registers (as packed fp32 pairs), so a product with the state is three shuffles away from complete and a token needs
+// no block-wide barrier.  The delta rule reads the state once per token and walks a prompt two tokens at a time, with
+// the small products between the two taken beforehand (A = S^T of the state before the pair):
+//   u_1 = b_1 (v_1 - w_1 A k_1),             o_1 = w_1 A q_1 + (k_1 . q_1) u_1
+//   u_2 = b_2 (v_2 - w_2 (w_1 A k_2 + (k_1 . k_2) u_1)),
+//   o_2 = w_2 (w_1 A q_2 + (k_1 . q_2) u_1) + (k_2 . q_2) u_2,        S <- w_2 (w_1 S + k_1 u_1^T) + k_2 u_2^T
+// so that the chain of dependent steps (products, shuffles, u, update) is paid once per pair.
+// Separate producer warps prepare the next block of tokens in shared memory (loads, unit length, the small products,
+// step size, decay) while the consumer warps walk the current one; one block-wide barrier per token block.  The state is stored
 // transposed, [v_dim][head_dim] per head, so that the eight lanes of a column read and write whole 128-byte lines.
 // Every output element is summed in one fixed order, so o does not depend on how a prompt was cut or batched.  A
 // request that starts at position 0 ignores what its state slots held before.
@@ -44,6 +48,11 @@ __device__ __forceinline__ float2 mul2(float2 a, float2 b) {
 __device__ __forceinline__ float hd_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float hd_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float hd_silu(float z) { return z / (1.0f + expf(-z)); }
+// the activations whose result is rounded to T: the fast exponential and division in 16-bit models
+template <typename T>
+__device__ __forceinline__ float silu_for(float z) { return silu_f32(z); }
+template <>
+__device__ __forceinline__ float silu_for<float>(float z) { return hd_silu(z); }
 
 // the rows a request brings: first position, first row of the batch, count; false: nothing to do
 struct RowSpan {
@@ -70,8 +79,22 @@ __device__ __forceinline__ bool row_span(RowSpan& s, int r, const int64_t* __res
   return s.n > 0 && s.pos0 >= 0;
 }
 
-template <typename T, int RPL, int TOK, int NPROD, int FORM>
-__global__ void __launch_bounds__((kHdConsumers + NPROD) * 32)
+// four elements of a row, kept as raw words between their load and their use
+template <typename T>
+struct alignas(4 * sizeof(T)) Quad {
+  uint32_t w[sizeof(T)];
+  __device__ __forceinline__ float get(int i) const {
+    if constexpr (sizeof(T) == 4) {
+      return __uint_as_float(w[i]);
+    } else {
+      const float2 f = unpack2<T>(w[i >> 1]);
+      return (i & 1) ? f.y : f.x;
+    }
+  }
+};
+
+template <typename T, int RPL, int TOK, int NPROD, int FORM, bool VEC>
+__global__ void __launch_bounds__((kHdConsumers + NPROD) * 32, RPL <= 16 && sizeof(T) == 2 ? 2 : 1)
 head_decay_kernel(float* __restrict__ o, const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v,
                   const T* __restrict__ z, const T* __restrict__ b, float* __restrict__ state,
                   const int64_t* __restrict__ req_pool_indices, const int64_t* __restrict__ seq_lens,
@@ -81,8 +104,6 @@ head_decay_kernel(float* __restrict__ o, const T* __restrict__ q, const T* __res
                   int64_t b_stride, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                   const float* __restrict__ skip, float q_scale, float unit_eps) {
   constexpr int DKP = RPL * 8;             // padded head_dim
-  constexpr int NE = (DKP + 31) / 32;      // elements per producer lane and row
-  constexpr int NB = TOK < 4 ? TOK : 4;    // tokens a producer warp loads at a time
   constexpr int BUF = TOK * (2 * DKP + kHdCols + 4);
   extern __shared__ __align__(16) float hd_smem[];  // (TOK > 1 ? 2 : 1) x { q | k [TOK][DKP], v [TOK][32], scalars [TOK][4] }
   griddep_wait();
@@ -93,75 +114,130 @@ head_decay_kernel(float* __restrict__ o, const T* __restrict__ q, const T* __res
   if (!row_span(sp, r, seq_lens, out_cache_loc, prefix_lens, extend_lens, extend_start_loc)) return;
   const int n = sp.n;
 
-  auto produce = [&](int t0, float* buf) {
-    const int pw = warp - kHdConsumers;
+  const int j = lane & 7;  // which eighth of the rows (chunks of four rows: j, j + 8, ...)
+  const float dt_bias_h = dt_bias[h], rate_h = expf(a_log[h]);
+  // Eight lanes prepare a token, a warp four tokens at a time, in ROUNDS rounds per block; tokens past the end become
+  // ones that change nothing.  The raw values of a block are loaded a whole block before they are prepared.
+  constexpr int ROUNDS = (TOK + 4 * NPROD - 1) / (4 * NPROD);
+  Quad<T> rq[ROUNDS][RPL / 4], rk[ROUNDS][RPL / 4], rv[ROUNDS];
+  T rz[ROUNDS], rb[ROUNDS];
+  auto load4 = [](const T* p, int d, int dim) {  // p[d .. d + 3], zeros from dim on
+    Quad<T> f;
+    if constexpr (VEC) {
+      f = d < dim ? *reinterpret_cast<const Quad<T>*>(p + d) : Quad<T>{};
+    } else {
+      float x[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[e] = d + e < dim ? to_f32<T>(p[d + e]) : 0.f;
+      if constexpr (sizeof(T) == 4) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) f.w[e] = __float_as_uint(x[e]);
+      } else {
+        f.w[0] = pack2<T>(x[0], x[1]);
+        f.w[1] = pack2<T>(x[2], x[3]);
+      }
+    }
+    return f;
+  };
+  auto fetch = [&](int t0) {
+    const int nt = n - t0 < TOK ? n - t0 : TOK;
+#pragma unroll
+    for (int x = 0; x < ROUNDS; ++x) {
+      const int tt = (x * NPROD + warp - kHdConsumers) * 4 + (lane >> 3);
+      const int64_t row = sp.row0 + t0 + (tt < nt ? tt : 0);
+#pragma unroll
+      for (int i = 0; i < RPL / 4; ++i) {
+        rq[x][i] = load4(q + row * q_stride + (int64_t)hk * dk, i * 32 + j * 4, dk);
+        rk[x][i] = load4(k + row * k_stride + (int64_t)hk * dk, i * 32 + j * 4, dk);
+      }
+      rv[x] = load4(v + row * v_stride + (int64_t)h * dv, col0 + j * 4, dv);
+      rz[x] = z[row * z_stride + h];
+      if (FORM == 1) rb[x] = b[row * b_stride + h];
+    }
+  };
+  auto prepare = [&](int t0, float* buf) {
     const int nt = n - t0 < TOK ? n - t0 : TOK;
     float* qs = buf;
     float* ks = qs + TOK * DKP;
     float* vs = ks + TOK * DKP;
     float* sc = vs + TOK * kHdCols;
-    for (int tb = pw * NB; tb < nt; tb += NPROD * NB) {
-      float qv[NB][NE], kv[NB][NE], vv[NB];
 #pragma unroll
-      for (int x = 0; x < NB; ++x) {
-        const bool ok = tb + x < nt;
-        const int64_t row = sp.row0 + t0 + (ok ? tb + x : tb);
+    for (int x = 0; x < ROUNDS; ++x) {
+      const int tt = (x * NPROD + warp - kHdConsumers) * 4 + (lane >> 3);
+      const bool ok = tt < nt;
+      float qv[RPL], kv[RPL], vv[4];
 #pragma unroll
-        for (int i = 0; i < NE; ++i) {
-          const int d = lane + 32 * i;
-          qv[x][i] = d < dk ? to_f32<T>(q[row * q_stride + (int64_t)hk * dk + d]) : 0.f;
-          kv[x][i] = d < dk ? to_f32<T>(k[row * k_stride + (int64_t)hk * dk + d]) : 0.f;
-        }
-        vv[x] = col0 + lane < dv ? to_f32<T>(v[row * v_stride + (int64_t)h * dv + col0 + lane]) : 0.f;
-      }
-      // lane x prepares the scalars of token tb + x
-      float w = 0.f, coef = 0.f;
-      if (lane < NB && tb + lane < nt) {
-        const int64_t row = sp.row0 + t0 + tb + lane;
-        const float dt = hd_softplus(to_f32<T>(z[row * z_stride + h]) + dt_bias[h]);
-        w = expf(-expf(a_log[h]) * dt);
-        coef = FORM == 0 ? dt : hd_sigmoid(to_f32<T>(b[row * b_stride + h]));
+      for (int i = 0; i < RPL; ++i) {
+        qv[i] = ok ? rq[x][i / 4].get(i % 4) : 0.f;
+        kv[i] = ok ? rk[x][i / 4].get(i % 4) : 0.f;
       }
 #pragma unroll
-      for (int x = 0; x < NB; ++x) {
-        float kq = 0.f;
-        if (FORM == 1) {
-          float sq = 0.f, sk = 0.f;
+      for (int i = 0; i < 4; ++i) vv[i] = rv[x].get(i);
+      const float dt = hd_softplus(to_f32<T>(rz[x]) + dt_bias_h);
+      const float w = ok ? expf(-rate_h * dt) : 1.f;
+      const float coef = !ok ? 0.f : FORM == 0 ? dt : hd_sigmoid(to_f32<T>(rb[x]));
+      float kq = 0.f, kk = 0.f, kn = 0.f;  // k . q, and for the second token of a pair k_first . k and k_first . q
+      if (FORM == 1) {
+        float sq = 0.f, sk = 0.f;
 #pragma unroll
-          for (int i = 0; i < NE; ++i) {
-            sq = fmaf(qv[x][i], qv[x][i], sq);
-            sk = fmaf(kv[x][i], kv[x][i], sk);
-            kq = fmaf(kv[x][i], qv[x][i], kq);
-          }
-          sq = warp_sum(sq);
-          sk = warp_sum(sk);
-          kq = warp_sum(kq);
-          const float fq = q_scale / sqrtf(sq + unit_eps), fk = 1.0f / sqrtf(sk + unit_eps);
-          kq *= fq * fk;
-#pragma unroll
-          for (int i = 0; i < NE; ++i) {
-            qv[x][i] *= fq;
-            kv[x][i] *= fk;
+        for (int i = 0; i < RPL; ++i) {
+          sq = fmaf(qv[i], qv[i], sq);
+          sk = fmaf(kv[i], kv[i], sk);
+          kq = fmaf(kv[i], qv[i], kq);
+          if (TOK > 1) {
+            const float kp = __shfl_xor_sync(0xffffffffu, kv[i], 8);  // the pair's other token
+            kk = fmaf(kp, kv[i], kk);
+            kn = fmaf(kp, qv[i], kn);
           }
         }
-        if (tb + x < nt) {
-          const int tt = tb + x;
 #pragma unroll
-          for (int i = 0; i < NE; ++i) {
-            const int d = lane + 32 * i;
-            qs[tt * DKP + d] = FORM == 0 ? qv[x][i] * q_scale : qv[x][i];
-            ks[tt * DKP + d] = kv[x][i];
+        for (int m = 1; m < 8; m <<= 1) {
+          sq += __shfl_xor_sync(0xffffffffu, sq, m);
+          sk += __shfl_xor_sync(0xffffffffu, sk, m);
+          kq += __shfl_xor_sync(0xffffffffu, kq, m);
+          if (TOK > 1) {
+            kk += __shfl_xor_sync(0xffffffffu, kk, m);
+            kn += __shfl_xor_sync(0xffffffffu, kn, m);
           }
-          vs[tt * kHdCols + lane] = vv[x];
-          if (lane == x) *reinterpret_cast<float4*>(sc + tt * 4) = make_float4(w, coef, kq, 0.f);
+        }
+        const float fq = q_scale / sqrtf(sq + unit_eps), fk = 1.0f / sqrtf(sk + unit_eps);
+        kq *= fq * fk;
+        if (TOK > 1) {
+          const float fp = __shfl_xor_sync(0xffffffffu, fk, 8);
+          kk *= fp * fk;
+          kn *= fp * fq;
+        }
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) {
+          qv[i] *= fq;
+          kv[i] *= fk;
+        }
+      } else if (q_scale != 1.f) {
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) qv[i] *= q_scale;
+      }
+      if (tt < TOK) {
+#pragma unroll
+        for (int i = 0; i < RPL / 4; ++i) {
+          const int d = tt * DKP + i * 32 + j * 4;
+          *reinterpret_cast<float4*>(qs + d) = make_float4(qv[4 * i], qv[4 * i + 1], qv[4 * i + 2], qv[4 * i + 3]);
+          *reinterpret_cast<float4*>(ks + d) = make_float4(kv[4 * i], kv[4 * i + 1], kv[4 * i + 2], kv[4 * i + 3]);
+        }
+        *reinterpret_cast<float4*>(vs + tt * kHdCols + j * 4) = make_float4(vv[0], vv[1], vv[2], vv[3]);
+        if (j == 0) {
+          *reinterpret_cast<float2*>(sc + tt * 4) = make_float2(w, coef);
+          sc[tt * 4 + 2] = kq;
+          if (FORM == 1 && (tt & 1)) {
+            sc[tt * 4 + 3] = kk;
+            sc[tt * 4 - 1] = kn;  // with the pair's first token: its k . q_next
+          }
         }
       }
     }
   };
 
   const bool producer = warp >= kHdConsumers;
-  const int j = lane & 7;                                      // which eighth of the rows
-  const int c = col0 + (producer ? 0 : warp) * 8 + (lane >> 3) * 2;  // this lane's columns c, c + 1
+  const int c = col0 + (producer ? 0 : warp) * 8 + (lane >> 3) * 2;  // a consumer lane's columns c, c + 1
   float* st = state + ((int64_t)req_pool_indices[r] * H + h) * (int64_t)dk * dv;
   const bool rows4 = (dk & 3) == 0;
   float2 S[2][RPL / 2];
@@ -187,7 +263,9 @@ head_decay_kernel(float* __restrict__ o, const T* __restrict__ q, const T* __res
         S[x][2 * i + 1] = make_float2(s4.z, s4.w);
       }
   } else {
-    produce(0, hd_smem);
+    fetch(0);
+    prepare(0, hd_smem);
+    if (TOK > 1 && TOK < n) fetch(TOK);
   }
   const float sk_h = (FORM == 0 && skip != nullptr) ? skip[h] : 0.f;
   __syncthreads();
@@ -195,13 +273,94 @@ head_decay_kernel(float* __restrict__ o, const T* __restrict__ q, const T* __res
   for (int t0 = 0; t0 < n; t0 += TOK) {
     float* buf = hd_smem + (TOK > 1 && ((t0 / TOK) & 1) ? BUF : 0);
     if (producer) {
-      if (TOK > 1 && t0 + TOK < n) produce(t0 + TOK, hd_smem + (((t0 / TOK) & 1) ? 0 : BUF));
+      if (TOK > 1 && t0 + TOK < n) {
+        prepare(t0 + TOK, hd_smem + (((t0 / TOK) & 1) ? 0 : BUF));
+        if (t0 + 2 * TOK < n) fetch(t0 + 2 * TOK);
+      }
     } else {
       const int nt = n - t0 < TOK ? n - t0 : TOK;
       const float* qs = buf;
       const float* ks = qs + TOK * DKP;
       const float* vs = ks + TOK * DKP;
       const float* sc = vs + TOK * kHdCols;
+      if (FORM == 1 && TOK > 1) {
+        constexpr bool HOLD = RPL <= 16;  // the pair's keys stay in registers between the two passes
+        for (int tt = 0; tt < nt; tt += 2) {
+          const float4* k4 = reinterpret_cast<const float4*>(ks + tt * DKP) + j;
+          const float4* q4 = reinterpret_cast<const float4*>(qs + tt * DKP) + j;
+          const float4 s1 = *reinterpret_cast<const float4*>(sc + tt * 4);      // w, b, k . q, k . q_next
+          const float4 s2 = *reinterpret_cast<const float4*>(sc + tt * 4 + 4);  // w, b, k . q, k . k_previous
+          const float2 v1 = *reinterpret_cast<const float2*>(vs + tt * kHdCols + warp * 8 + (lane >> 3) * 2);
+          const float2 v2 = *reinterpret_cast<const float2*>(vs + (tt + 1) * kHdCols + warp * 8 + (lane >> 3) * 2);
+          float2 kr[2][HOLD ? RPL / 2 : 1];
+          float2 acc[8];  // k_1, k_2, q_1, q_2 by column
+#pragma unroll
+          for (int i = 0; i < 8; ++i) acc[i] = make_float2(0.f, 0.f);
+#pragma unroll
+          for (int i = 0; i < RPL / 4; ++i) {
+            const float4 f[4] = {k4[i * 8], k4[i * 8 + DKP / 4], q4[i * 8], q4[i * 8 + DKP / 4]};
+#pragma unroll
+            for (int y = 0; y < 4; ++y) {
+              const float2 lo = make_float2(f[y].x, f[y].y), hi = make_float2(f[y].z, f[y].w);
+              if (HOLD && y < 2) { kr[y][2 * i] = lo; kr[y][2 * i + 1] = hi; }
+              acc[2 * y] = fma2(S[0][2 * i], lo, acc[2 * y]);
+              acc[2 * y + 1] = fma2(S[1][2 * i], lo, acc[2 * y + 1]);
+              acc[2 * y] = fma2(S[0][2 * i + 1], hi, acc[2 * y]);
+              acc[2 * y + 1] = fma2(S[1][2 * i + 1], hi, acc[2 * y + 1]);
+            }
+          }
+          // sum over the eight lanes; lane j ends with value j
+          float p[8], t4[4], t2[2];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) p[i] = acc[i].x + acc[i].y;
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float got = __shfl_xor_sync(0xffffffffu, (j & 4) ? p[i] : p[i + 4], 4);
+            t4[i] = ((j & 4) ? p[i + 4] : p[i]) + got;
+          }
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const float got = __shfl_xor_sync(0xffffffffu, (j & 2) ? t4[i] : t4[i + 2], 2);
+            t2[i] = ((j & 2) ? t4[i + 2] : t4[i]) + got;
+          }
+          const float got = __shfl_xor_sync(0xffffffffu, (j & 1) ? t2[0] : t2[1], 1);
+          const float mine = ((j & 1) ? t2[1] : t2[0]) + got;
+          const int g0 = lane & 24;  // the eight lanes' first
+          const float a10 = __shfl_sync(0xffffffffu, mine, g0), a11 = __shfl_sync(0xffffffffu, mine, g0 + 1);
+          const float a20 = __shfl_sync(0xffffffffu, mine, g0 + 2), a21 = __shfl_sync(0xffffffffu, mine, g0 + 3);
+          const float u10 = s1.y * (v1.x - s1.x * a10), u11 = s1.y * (v1.y - s1.x * a11);
+          const float u20 = s2.y * (v2.x - s2.x * fmaf(s2.w, u10, s1.x * a20));
+          const float u21 = s2.y * (v2.y - s2.x * fmaf(s2.w, u11, s1.x * a21));
+          if (j >= 4) {  // lanes 4 - 7 hold the products with q_1 (two columns), q_2 (two columns)
+            const float u1 = (j & 1) ? u11 : u10, u2 = (j & 1) ? u21 : u20;
+            const float first = s1.x * mine;
+            const float out = (j & 2) ? fmaf(s2.z, u2, s2.x * fmaf(s1.w, u1, first)) : fmaf(s1.z, u1, first);
+            const int tok = tt + ((j >> 1) & 1), col = c + (j & 1);
+            if (tok < nt && col < dv) o[((sp.row0 + t0 + tok) * H + h) * (int64_t)dv + col] = out;
+          }
+          const float w12 = s1.x * s2.x;
+          const float2 wp = make_float2(w12, w12);
+          const float2 x10 = make_float2(s2.x * u10, s2.x * u10), x11 = make_float2(s2.x * u11, s2.x * u11);
+          const float2 x20 = make_float2(u20, u20), x21 = make_float2(u21, u21);
+#pragma unroll
+          for (int i = 0; i < RPL / 4; ++i) {
+            float2 ka[2], kb[2];
+            if (HOLD) {
+              ka[0] = kr[0][HOLD ? 2 * i : 0]; ka[1] = kr[0][HOLD ? 2 * i + 1 : 0];
+              kb[0] = kr[1][HOLD ? 2 * i : 0]; kb[1] = kr[1][HOLD ? 2 * i + 1 : 0];
+            } else {
+              const float4 f = k4[i * 8], e = k4[i * 8 + DKP / 4];
+              ka[0] = make_float2(f.x, f.y); ka[1] = make_float2(f.z, f.w);
+              kb[0] = make_float2(e.x, e.y); kb[1] = make_float2(e.z, e.w);
+            }
+#pragma unroll
+            for (int y = 0; y < 2; ++y) {
+              S[0][2 * i + y] = fma2(kb[y], x20, fma2(ka[y], x10, mul2(wp, S[0][2 * i + y])));
+              S[1][2 * i + y] = fma2(kb[y], x21, fma2(ka[y], x11, mul2(wp, S[1][2 * i + y])));
+            }
+          }
+        }
+      } else
       for (int tt = 0; tt < nt; ++tt) {
         const float4* k4 = reinterpret_cast<const float4*>(ks + tt * DKP) + j;
         const float4* q4 = reinterpret_cast<const float4*>(qs + tt * DKP) + j;
@@ -297,7 +456,7 @@ head_decay_kernel(float* __restrict__ o, const T* __restrict__ q, const T* __res
   }
 }
 
-template <typename T, int RPL, int TOK, int NPROD, int FORM>
+template <typename T, int RPL, int TOK, int NPROD, int FORM, bool VEC>
 int head_decay_launch(dim3 grid, cudaStream_t stream, float* o, const void* q, const void* k, const void* v,
                       const void* z, const void* b, float* state, const int64_t* req_pool_indices,
                       const int64_t* seq_lens, const int64_t* out_cache_loc, const int32_t* prefix_lens,
@@ -307,11 +466,11 @@ int head_decay_launch(dim3 grid, cudaStream_t stream, float* o, const void* q, c
   const size_t smem = sizeof(float) * (TOK > 1 ? 2 : 1) * (size_t)TOK * (2 * RPL * 8 + kHdCols + 4);
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
-    SPD_CUDA(cudaFuncSetAttribute(head_decay_kernel<T, RPL, TOK, NPROD, FORM>,
+    SPD_CUDA(cudaFuncSetAttribute(head_decay_kernel<T, RPL, TOK, NPROD, FORM, VEC>,
                                   cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = smem;
   }
-  SPD_CUDA(launch(head_decay_kernel<T, RPL, TOK, NPROD, FORM>, grid, dim3((kHdConsumers + NPROD) * 32), smem, stream,
+  SPD_CUDA(launch(head_decay_kernel<T, RPL, TOK, NPROD, FORM, VEC>, grid, dim3((kHdConsumers + NPROD) * 32), smem, stream,
                   pdl_enabled(), o, (const T*)q, (const T*)k, (const T*)v, (const T*)z, (const T*)b, state,
                   req_pool_indices, seq_lens, out_cache_loc, prefix_lens, extend_lens, extend_start_loc, H, Hk, dk, dv,
                   q_stride, k_stride, v_stride, z_stride, b_stride, dt_bias, a_log, skip, q_scale, unit_eps));
@@ -324,8 +483,8 @@ int head_decay_launch(dim3 grid, cudaStream_t stream, float* o, const void* q, c
 // first; zeros at position 0); the slot then receives its last TAPS - 1 inputs.  One CTA per (request, slice of the
 // channels, chunk of the request's rows); the CTA of the first chunk is the only one that touches the slot.
 // ------------------------------------------------------------------------------------------------
-constexpr int kConvThreads = 128;
-constexpr int kConvChunk = 32;
+constexpr int kConvThreads = 128;  // at most
+constexpr int kConvChunk = 16;
 constexpr int kConvMaxTaps = 8;
 
 template <typename T, int VEC, int TAPS>
@@ -339,7 +498,7 @@ short_conv_kernel(T* __restrict__ out, const T* __restrict__ x, const T* __restr
   griddep_launch_dependents();
   constexpr int HIST = TAPS - 1;
   const int r = blockIdx.x;
-  const int64_t c = ((int64_t)blockIdx.y * kConvThreads + threadIdx.x) * VEC;
+  const int64_t c = ((int64_t)blockIdx.y * blockDim.x + threadIdx.x) * VEC;
   if (c >= channels) return;
   RowSpan sp;
   if (!row_span(sp, r, seq_lens, out_cache_loc, prefix_lens, extend_lens, extend_start_loc)) return;
@@ -403,7 +562,7 @@ short_conv_kernel(T* __restrict__ out, const T* __restrict__ x, const T* __restr
 #pragma unroll
       for (int e = 0; e < VEC; ++e) y[e] = fmaf(wt[i][e], hist[i][e], y[e]);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) y[e] = hd_silu(fmaf(wt[HIST][e], cur[e], y[e]));
+    for (int e = 0; e < VEC; ++e) y[e] = silu_for<T>(fmaf(wt[HIST][e], cur[e], y[e]));
 #pragma unroll
     for (int i = 0; i + 1 < HIST; ++i)
 #pragma unroll
@@ -429,11 +588,13 @@ int short_conv_launch(int64_t batch, int64_t rows, cudaStream_t stream, void* ou
                       const void* bias, float* conv_state, const int64_t* req_pool_indices, const int64_t* seq_lens,
                       const int64_t* out_cache_loc, const int32_t* prefix_lens, const int32_t* extend_lens,
                       const int32_t* extend_start_loc, int64_t channels, int64_t x_stride) {
-  const int64_t per = (int64_t)kConvThreads * VEC;
+  // whole warps, the channels spread evenly over the fewest CTAs
+  const int64_t vecs = (channels + VEC - 1) / VEC, ctas = (vecs + kConvThreads - 1) / kConvThreads;
+  const int64_t threads = ((vecs + ctas - 1) / ctas + 31) / 32 * 32, per = threads * VEC;
   const int64_t chunks = (rows + kConvChunk - 1) / kConvChunk;
   SPD_REQUIRE(chunks <= 65535 && (channels + per - 1) / per <= 65535, SPD_E_SHAPE, "spd_short_conv: too many rows or channels");
   const dim3 grid((unsigned)batch, (unsigned)((channels + per - 1) / per), (unsigned)chunks);
-  SPD_CUDA(launch(short_conv_kernel<T, VEC, TAPS>, grid, dim3(kConvThreads), 0, stream, pdl_enabled(), (T*)out,
+  SPD_CUDA(launch(short_conv_kernel<T, VEC, TAPS>, grid, dim3((unsigned)threads), 0, stream, pdl_enabled(), (T*)out,
                   (const T*)x, (const T*)w, (const T*)bias, conv_state, req_pool_indices, seq_lens, out_cache_loc,
                   prefix_lens, extend_lens, extend_start_loc, channels, x_stride));
   return 0;
@@ -524,18 +685,23 @@ int spd_head_decay(float* o, const void* q, const void* k, const void* v, const 
   grid, as_stream(stream), o, q, k, v, z, b, state, req_pool_indices, seq_lens, out_cache_loc, prefix_lens,          \
       extend_lens, extend_start_loc, num_heads, num_k_heads, head_dim, v_dim, q_stride, k_stride, v_stride, z_stride, \
       b_stride, dt_bias, a_log, skip, q_scale, unit_eps
-#define SPD_HD_SHAPE(RPL)                                                                    \
-  do {                                                                                       \
-    if (decode) return form == 0 ? head_decay_launch<T, RPL, 1, 1, 0>(SPD_HD_ARGS)           \
-                                 : head_decay_launch<T, RPL, 1, 1, 1>(SPD_HD_ARGS);          \
-    return form == 0 ? head_decay_launch<T, RPL, kHdTok, 2, 0>(SPD_HD_ARGS)                  \
-                     : head_decay_launch<T, RPL, kHdTok, 2, 1>(SPD_HD_ARGS);                 \
+#define SPD_HD_SHAPE(RPL, VEC)                                                                    \
+  do {                                                                                            \
+    if (decode) return form == 0 ? head_decay_launch<T, RPL, 1, 1, 0, VEC>(SPD_HD_ARGS)           \
+                                 : head_decay_launch<T, RPL, 1, 1, 1, VEC>(SPD_HD_ARGS);          \
+    return form == 0 ? head_decay_launch<T, RPL, kHdTok, 2, 0, VEC>(SPD_HD_ARGS)                  \
+                     : head_decay_launch<T, RPL, kHdTok, 2, 1, VEC>(SPD_HD_ARGS);                 \
   } while (0)
   SPD_DISPATCH_ANY(dtype, {
-    if (head_dim <= 32) SPD_HD_SHAPE(4);
-    else if (head_dim <= 64) SPD_HD_SHAPE(8);
-    else if (head_dim <= 128) SPD_HD_SHAPE(16);
-    else SPD_HD_SHAPE(32);
+    // rows in groups of four elements; other sizes take one element-wise instantiation
+    const bool vec = ((head_dim | v_dim | q_stride | k_stride | v_stride) & 3) == 0 &&
+                     ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) &
+                      (sizeof(Quad<T>) - 1)) == 0;
+    if (!vec) SPD_HD_SHAPE(32, false);
+    else if (head_dim <= 32) SPD_HD_SHAPE(4, true);
+    else if (head_dim <= 64) SPD_HD_SHAPE(8, true);
+    else if (head_dim <= 128) SPD_HD_SHAPE(16, true);
+    else SPD_HD_SHAPE(32, true);
   });
 #undef SPD_HD_SHAPE
 #undef SPD_HD_ARGS

@@ -222,7 +222,101 @@ rotary_segments_vec_kernel(RotarySegments segs, const int64_t* __restrict__ posi
   }
 }
 
-// The form with per-head norms: a warp per (token, head), the head's channels in shared memory between the norm and
+// The form with per-head norms in 16-byte pieces (every segment turns whole heads or none in the half-split layout, its
+// head_dim / (2 N) is a power of two of at most 32, strides and pointers aligned): a lane owns vector i of a head's
+// first half and vector i of its second half — rotation partners — and the head's lanes sum their squares by shuffles.
+// The items (lane, head) of all segments form one list, each segment starting at a warp boundary.
+template <typename T>
+__global__ void __launch_bounds__(256)
+rotary_segments_norm_vec_kernel(RotarySegments segs, const int64_t* __restrict__ positions,
+                                const int64_t* __restrict__ loc, const float* __restrict__ cos_sin, int rot_max,
+                                int64_t max_positions) {
+  griddep_wait();
+  griddep_launch_dependents();
+  constexpr int N = Vec16<T>::kN;
+  const int64_t t = blockIdx.x;
+  int64_t p = positions[t];
+  p = p < 0 ? 0 : (p < max_positions ? p : max_positions - 1);
+  const float* cs = cos_sin != nullptr ? cos_sin + p * rot_max : nullptr;
+  const int half_max = rot_max >> 1;
+  const int64_t slot = loc != nullptr ? loc[t] : 0;
+  int total = 0;
+  for (int sidx = 0; sidx < segs.n; ++sidx) total += (segs.seg[sidx].heads * (segs.seg[sidx].head_dim / (2 * N)) + 31) & ~31;
+  for (int it = threadIdx.x; it < total; it += blockDim.x) {  // uniform over a warp
+    int sidx = 0, item = it;
+    for (;; ++sidx) {
+      const int n = (segs.seg[sidx].heads * (segs.seg[sidx].head_dim / (2 * N)) + 31) & ~31;
+      if (item < n) break;
+      item -= n;
+    }
+    const RotarySegment& sg = segs.seg[sidx];
+    const int gl = sg.head_dim / (2 * N), half = sg.head_dim >> 1;
+    const int h = item / gl, d0 = (item - h * gl) * N;
+    const bool on = h < sg.heads;
+    const T* sp = reinterpret_cast<const T*>(sg.src) + t * sg.src_row + (on ? h : 0) * sg.src_head + d0;
+    const Vec16<T> va = ldv(sp), vb = ldv(sp + half);
+    float a[N], b[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      a[i] = to_f32<T>(va.e()[i]);
+      b[i] = to_f32<T>(vb.e()[i]);
+    }
+    auto with4 = [&](const float* src, bool add) {  // add to / multiply by the head's fp32 vector
+#pragma unroll
+      for (int i = 0; i < N; i += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(src + d0 + i), y = *reinterpret_cast<const float4*>(src + half + d0 + i);
+        if (add) {
+          a[i] += x.x; a[i + 1] += x.y; a[i + 2] += x.z; a[i + 3] += x.w;
+          b[i] += y.x; b[i + 1] += y.y; b[i + 2] += y.z; b[i + 3] += y.w;
+        } else {
+          a[i] *= x.x; a[i + 1] *= x.y; a[i + 2] *= x.z; a[i + 3] *= x.w;
+          b[i] *= y.x; b[i + 1] *= y.y; b[i + 2] *= y.z; b[i + 3] *= y.w;
+        }
+      }
+    };
+    if (sg.bias != nullptr) with4(sg.bias + (on ? h : 0) * sg.head_dim, true);
+    if (sg.norm) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) ss = fmaf(a[i], a[i], fmaf(b[i], b[i], ss));
+      for (int m = 1; m < gl; m <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+      const float inv = 1.0f / sqrtf(ss / (float)sg.head_dim + sg.norm_eps);
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        a[i] *= inv;
+        b[i] *= inv;
+      }
+      if (sg.norm_w != nullptr) with4(sg.norm_w, false);
+    }
+    if (sg.rot) {
+#pragma unroll
+      for (int i = 0; i < N; i += 4) {
+        const float4 c4 = *reinterpret_cast<const float4*>(cs + d0 + i);
+        const float4 s4 = *reinterpret_cast<const float4*>(cs + half_max + d0 + i);
+        const float c[4] = {c4.x, c4.y, c4.z, c4.w}, sn[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float x = a[i + e], y = b[i + e];
+          a[i + e] = x * c[e] - y * sn[e];
+          b[i + e] = y * c[e] + x * sn[e];
+        }
+      }
+    }
+    if (on) {
+      T* dp = reinterpret_cast<T*>(sg.dst) + (sg.to_pool ? slot : t) * sg.dst_row + h * sg.dst_head + d0;
+      Vec16<T> oa, ob;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        oa.e()[i] = from_f32<T>(a[i]);
+        ob.e()[i] = from_f32<T>(b[i]);
+      }
+      stv(dp, oa);
+      stv(dp + half, ob);
+    }
+  }
+}
+
+// The same for any sizes and either layout: a warp per (token, head), the head's channels in shared memory between the norm and
 // the rotation.  VEC consecutive channels per lane and step (head_dim a multiple of 32 VEC for every segment, rows and
 // heads aligned to VEC elements), else VEC = 1.
 constexpr int kRotNormMaxDim = 512;
@@ -557,6 +651,25 @@ int spd_rotary_segments(const spd_rotary_segment_t* segments, int num_segments, 
     SPD_REQUIRE(dim_max <= kRotNormMaxDim, SPD_E_SHAPE, "spd_rotary_segments: normed heads of %d channels (max %d)",
                 dim_max, kRotNormMaxDim);
     const int pad = (dim_max + 3) / 4 * 4;
+    const int nv = dtype == SPD_F32 ? 4 : 8;
+    bool pieces = !paired && rot_max % 8 == 0 && aligned16(cos_sin);
+    int items = 0;
+    for (int i = 0; i < num_segments; ++i) {
+      const RotarySegment& s = segs.seg[i];
+      const int gl = s.head_dim / (2 * nv);
+      pieces = pieces && s.head_dim % (2 * nv) == 0 && gl <= 32 && (gl & (gl - 1)) == 0 && (s.rot == 0 || s.rot == s.head_dim) &&
+               s.src_head % nv == 0 && s.dst_head % nv == 0 && s.src_row % nv == 0 && s.dst_row % nv == 0 &&
+               aligned16(s.src) && aligned16(s.dst) && aligned16(s.bias) && aligned16(s.norm_w);
+      items += (s.heads * gl + 31) / 32 * 32;
+    }
+    if (pieces) {
+      const int threads = items < 256 ? items : 256;
+      SPD_DISPATCH_ANY(dtype, {
+        SPD_CUDA(launch(rotary_segments_norm_vec_kernel<T>, dim3((unsigned)tokens), dim3((unsigned)threads), 0,
+                        as_stream(stream), pdl_enabled(), segs, positions, loc, cos_sin, rot_max, max_positions));
+      });
+      return 0;
+    }
     SPD_DISPATCH_ANY(dtype, {
       auto kern = step == 4   ? rotary_segments_norm_kernel<T, 4>
                   : step == 2 ? rotary_segments_norm_kernel<T, 2>
