@@ -473,8 +473,8 @@ kv_store_kernel(const T* __restrict__ k, const T* __restrict__ v, T* __restrict_
 }
 
 // Block rows of the blocks that a batch completes: the mean over the block's cache rows of K and V, as the cache holds
-// them, in fp32.  One CTA per (request, block that its new tokens may complete); a row's vectors (K, then V) go to
-// neighbouring threads, and where they leave threads over, TL of them share a vector by tokens (their sums meet in
+// them, in fp32.  One CTA per (request, block that its new tokens may complete, slice of the row); a row's vectors (K,
+// then V) go to neighbouring threads, and where they leave threads over, TL of them share a vector by tokens (their sums meet in
 // shared memory, in a fixed order).
 constexpr int kPoolThreads = 128;
 constexpr int kPoolSlots = 512;  // slot numbers staged at a time
@@ -501,7 +501,7 @@ pool_key_blocks_kernel(T* __restrict__ k_pool, T* __restrict__ v_pool, const int
   const int per = kPoolThreads / tl_lanes;  // vectors in flight
   const int tl = threadIdx.x / per, lv = threadIdx.x - tl * per;
   const int64_t kv = k_row / VEC, nv = kv + (v_pool != nullptr ? v_row / VEC : 0);
-  for (int64_t v0 = 0; v0 < nv; v0 += per) {
+  for (int64_t v0 = (int64_t)blockIdx.z * per; v0 < nv; v0 += (int64_t)gridDim.z * per) {
     const int64_t v = v0 + lv;
     const bool on = tl < tl_lanes && v < nv;
     T* pool = v < kv ? k_pool : v_pool;
@@ -599,7 +599,7 @@ int spd_pool_key_blocks(void* k_pool, void* v_pool, const int32_t* req_to_token,
   if (batch == 0 || rows <= 0) return 0;
   SPD_REQUIRE(batch <= 65535, SPD_E_SHAPE, "spd_pool_key_blocks: batch too large");
   const KeyBlocks kb{block_size, block_run_len, (block_run_len + block_size - 1) / block_size, block_base};
-  const dim3 grid((unsigned)((rows + block_size - 1) / block_size), (unsigned)batch);  // n new tokens complete at most that many
+  const int64_t blocks = (rows + block_size - 1) / block_size;  // n new tokens complete at most that many
   SPD_DISPATCH_ANY(dtype, {
     constexpr int N = 16 / (int)sizeof(T);
     const bool vec = k_row_elems % N == 0 && v_row_elems % N == 0 && aligned16(k_pool) && aligned16(v_pool);
@@ -607,6 +607,9 @@ int spd_pool_key_blocks(void* k_pool, void* v_pool, const int32_t* req_to_token,
     const int64_t vecs = (k_row_elems + (v_pool != nullptr ? v_row_elems : 0)) / (vec ? N : 1);
     int tl = 1;  // token lanes per vector
     while (tl < 8 && tl * 2 <= block_size && vecs * tl * 2 <= kPoolThreads) tl *= 2;
+    if (tl == 1 && block_size >= 8) tl = 2;
+    const int64_t slices = (vecs * tl + kPoolThreads - 1) / kPoolThreads;
+    const dim3 grid((unsigned)blocks, (unsigned)batch, (unsigned)(slices < 64 ? slices : 64));
     SPD_CUDA(launch(kern, grid, dim3(kPoolThreads), 0, as_stream(stream), pdl_enabled(), (T*)k_pool, (T*)v_pool,
                     req_to_token, req_pool_indices, seq_lens, prefix_lens, extend_lens, req_to_token_stride, k_row_elems,
                     v_row_elems, tl, kb));

@@ -86,21 +86,33 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
   // the tile's keys in one list: the NB blocks its last row sees, then the tokens j_lo .. j_hi
   const int NB = (int)key_blocks_seen(kb, j_hi, window), n_keys = NB + (int)(j_hi - j_lo) + 1;
   const int ntiles = (n_keys - 1) / kGmBK + 1;
-  auto load_kv = [&](int t, int buf) {
-    const int eb = t * kGmBK;
-    for (int idx = tid; idx < kGmBK * (DK / 8); idx += kGmThreads) {
-      const int row = idx / (DK / 8), c = idx % (DK / 8);
-      const bool ok = eb + row < n_keys;
-      const int64_t slot = ok ? key_row(kb, page, eb + row, NB, j_lo) : 0;
-      cp_async16(smem_u32(sK + (buf * kGmBK + row) * LDK + c * 8), k_pool + (slot * G + g) * DK + c * 8, ok);
-    }
-    for (int idx = tid; idx < kGmBK * (DV / 8); idx += kGmThreads) {
-      const int row = idx / (DV / 8), c = idx % (DV / 8);
-      const bool ok = eb + row < n_keys;
-      const int64_t slot = ok ? key_row(kb, page, eb + row, NB, j_lo) : 0;
-      cp_async16(smem_u32(sV + (buf * kGmBK + row) * LDV + c * 8), v_pool + slot * v_slot + (int64_t)(g % Gv) * DV + c * 8, ok);
+  // pool rows of a tile's keys (-1 past the end), found two tiles ahead of their use
+  __shared__ int slots[2][kGmBK];
+  auto find_rows = [&](int t) {
+    if (tid < kGmBK) {
+      const int e = t * kGmBK + tid;
+      slots[t & 1][tid] = e < n_keys ? key_row(kb, page, e, NB, j_lo) : -1;
     }
   };
+  auto load_kv = [&](int t, int buf) {
+    const int* row_of = slots[t & 1];
+#pragma unroll 4
+    for (int idx = tid; idx < kGmBK * (DK / 8); idx += kGmThreads) {
+      const int row = idx / (DK / 8), c = idx % (DK / 8);
+      const int64_t slot = row_of[row];
+      cp_async16(smem_u32(sK + (buf * kGmBK + row) * LDK + c * 8), k_pool + ((slot < 0 ? 0 : slot) * G + g) * DK + c * 8, slot >= 0);
+    }
+#pragma unroll 4
+    for (int idx = tid; idx < kGmBK * (DV / 8); idx += kGmThreads) {
+      const int row = idx / (DV / 8), c = idx % (DV / 8);
+      const int64_t slot = row_of[row];
+      cp_async16(smem_u32(sV + (buf * kGmBK + row) * LDV + c * 8),
+                 v_pool + (slot < 0 ? 0 : slot) * v_slot + (int64_t)(g % Gv) * DV + c * 8, slot >= 0);
+    }
+  };
+  find_rows(0);
+  find_rows(1);
+  __syncthreads();
   load_kv(0, 0);
   cp_async_commit();
 
@@ -143,6 +155,7 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
       cp_async_wait<0>();
     }
     __syncthreads();
+    if (t + 2 < ntiles) find_rows(t + 2);  // (tile t's list has been read; the barrier at the end publishes this one)
     float s[kGmBK / 8][4];
 #pragma unroll
     for (int i = 0; i < kGmBK / 8; ++i)
