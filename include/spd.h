@@ -161,7 +161,8 @@ int spd_bias_act_residual(void* out, const void* x, const void* bias, const void
  * fp32 accumulator itself (routers and logits of models that want them in 32-bit).
  * epilogue: SPD_EPI_NONE, or SPD_EPI_SILU_MUL: W is [2N, K] (gate rows || up rows, the
  * MergedColumnParallelLinear order, S/models/llama.py:67-73) and C[M,N] = silu(A Wg^T) * (A Wu^T),
- * both products rounded to dtype first (== gate_up_proj followed by SiluAndMul).
+ * both products rounded to dtype first (== gate_up_proj followed by SiluAndMul), or SPD_EPI_GELU: C =
+ * gelu(A W^T), the erf form of the product rounded to dtype (M > 256 only; out_f32 0).
  * workspace: device scratch for the stream-K partials and their "published" flags
  * (spd_gemm_workspace_bytes()), zero-initialised ONCE by the caller and then owned by one stream
  * (the kernels re-arm the flags themselves; two streams must not share one workspace).  May be
@@ -171,6 +172,7 @@ int spd_bias_act_residual(void* out, const void* x, const void* bias, const void
  * ------------------------------------------------------------------------------------------- */
 #define SPD_EPI_NONE 0
 #define SPD_EPI_SILU_MUL 1
+#define SPD_EPI_GELU 2
 int64_t spd_gemm_workspace_bytes(void);
 int spd_gemm(void* C, const void* A, const void* W, int64_t M, int64_t N, int64_t K, int64_t lda,
              int64_t ldw, int64_t ldc, int dtype, int out_f32, int epilogue, void* workspace,
@@ -286,7 +288,7 @@ int spd_comm_destroy(spd_comm_t* comm);
  *   expert in 128-row tiles (spd_moe_align / spd_moe_gather), tile_group[i] = expert of rows
  *   [128 i, 128 i + 128) or < 0 (unused tile, skipped); W = the experts' weights stacked,
  *   [num_groups * N, K] — with SPD_EPI_SILU_MUL [num_groups * 2N, K], gate rows || up rows per expert;
- *   C [M, N].  a_group_stride must be 0.
+ *   C [M, N].  a_group_stride must be 0.  SPD_EPI_GELU: the erf-form GELU of the products (stacked weights).
  * cols mode (tile_group == NULL) — block-diagonal products, the absorbed-MLA BMMs
  *   torch.bmm(q_nope, w_kc) / torch.bmm(attn_out, w_vc) (S/models/deepseek_v2.py:667,702):
  *   C[:, g*N:(g+1)*N] = A[:, g*a_group_stride : g*a_group_stride + K] * W[g*N:(g+1)*N, :K]^T,
@@ -377,21 +379,25 @@ int spd_linear_simt(void* C, const void* A, const void* W, int64_t M, int64_t N,
  * the top_k largest scores are chosen (ties: smaller expert id), weights = score (renormalised over the
  * chosen ones if renormalize) x scale.
  * correction (fp32 [experts], nullable) biases the SELECTION only (weights stay unbiased).  num_groups > 1: the
- * experts are cut into equal runs of neighbours, a run ranks by its top-2 biased scores added together, and
- * selection is restricted to the keep_groups highest-ranked runs. */
+ * experts are cut into equal runs of neighbours, a run ranks by its largest biased score (group_top 1) or its two
+ * largest added together (2), and selection is restricted to the keep_groups highest-ranked runs. */
 int spd_moe_route_scores(int32_t* topk_ids, float* topk_w, const float* logits, int64_t ld, int64_t tokens,
                          int num_experts, int top_k, int score_func, int renormalize, float scale,
-                         const float* correction, int num_groups, int keep_groups, spd_stream_t stream);
+                         const float* correction, int num_groups, int keep_groups, int group_top,
+                         spd_stream_t stream);
 /* xs[r, :] = w(r) * x[row_token[r], :] with w(r) the routing weight of the entry sorted to row r (1 if
  * topk_w == NULL); zeros for padding rows — experts that weight their INPUT */
 int spd_moe_gather_scaled(void* xs, const void* x, const int32_t* row_token, const int32_t* inv_pos,
                           const float* topk_w, int64_t rows, int top_k, int64_t dim, int64_t x_stride,
                           int dtype, spd_stream_t stream);
 /* out[t, :] = sum_j (topk_w ? topk_w[t, j] : 1) * y[inv_pos[t * top_k + j], :]
- *           + (shared ? (shared_gate ? sigmoid(shared_gate[t * gate_stride]) : 1) * shared[t, :] : 0) */
+ *           + (shared ? (shared_gate ? sigmoid(shared_gate[t * gate_stride]) : 1) * shared[t, :] : 0)
+ * An entry with inv_pos < 0 (spd_moe_align: a choice outside the experts) contributes row t of `input` (row stride
+ * input_stride) instead of a row of y — an expert that hands its input on —, or nothing where input is NULL. */
 int spd_moe_combine_gated(void* out, const void* y, const int32_t* inv_pos, const float* topk_w,
-                          const void* shared, const float* shared_gate, int64_t gate_stride, int64_t tokens,
-                          int top_k, int64_t dim, int dtype, spd_stream_t stream);
+                          const void* shared, const float* shared_gate, int64_t gate_stride, const void* input,
+                          int64_t input_stride, int64_t tokens, int top_k, int64_t dim, int dtype,
+                          spd_stream_t stream);
 /* k_pool[loc[t]] = k[t], v_pool[loc[t]] = v[t] with different row sizes for keys and values */
 int spd_kv_store(const void* k, const void* v, void* k_pool, void* v_pool, const int64_t* loc,
                  int64_t tokens, int64_t k_row_elems, int64_t v_row_elems, int64_t k_stride,
@@ -467,7 +473,7 @@ int spd_embed_sincos(float* x, const void* table, const int64_t* idx, const int6
 /* out[r, :] = [a[r, :] | b[r, :]] converted to dtype (a, b fp32 [rows, dim]; out [rows, 2 dim]) */
 int spd_cast_concat(void* out, const float* a, const float* b, int64_t rows, int64_t dim, int dtype,
                     spd_stream_t stream);
-/* out[r, c] = act(x[r * x_stride + c]); act 0 SiLU, 1 tanh-form GELU, 2 relu squared, 3 tanh, 4 relu */
+/* out[r, c] = act(x[r * x_stride + c]); act 0 SiLU, 1 tanh-form GELU, 2 relu squared, 3 tanh, 4 relu, 5 erf-form GELU */
 int spd_activation(void* out, const void* x, int64_t rows, int64_t cols, int64_t x_stride, int act, int dtype,
                    spd_stream_t stream);
 /* y = x[r, :dim] / sqrt(mean(x[r, :dim]^2) + eps) * w; pool[loc[r] * pool_stride + :] = y (pool nullable) and
@@ -568,9 +574,10 @@ typedef struct {
   void* dst;
   int64_t src_row, dst_row;
   int32_t heads, head_dim, rot, src_head, dst_head, to_pool;
-  const float* norm_w;  /* norm != 0: after the bias and before the rotation the head is brought to unit RMS over its */
+  const float* norm_w;  /* norm 1: after the bias and before the rotation the head is brought to unit RMS over its */
   int32_t norm;         /* head_dim channels (norm_eps inside the root) and multiplied by norm_w (fp32 [head_dim], */
-  float norm_eps;       /* shared by the heads; NULL: no weight).  At most 512 channels then. */
+  float norm_eps;       /* shared by the heads; NULL: no weight); at most 512 channels then.  norm 2: unit RMS over all */
+                        /* heads of the segment together, norm_w fp32 [heads * head_dim]; not beside norm 1 segments. */
 } spd_rotary_segment_t;
 /* Up to four segments in one launch.  cos_sin fp32 [max_positions, rot_max] = cos || sin (rot_max / 2 each) of
  * position * f_i; a segment with rot < rot_max uses the first rot / 2 of both.  paired != 0: channel 2 i turns
@@ -611,6 +618,19 @@ int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const 
                             int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
                             int64_t v_slot_stride, int block_size, int block_run_len, int64_t block_base, int dtype,
                             spd_stream_t stream);
+/* spd_attn_general_blocks with two more options.  keep_first > 0 (with a window, without blocks): positions 0 ..
+ * keep_first - 1 of a request stay visible when the window has moved past them, at their true distance.  dist_bias
+ * (fp32 [num_q_heads, dist_bias_len], nullable, without blocks): dist_bias[h, min(i - j, dist_bias_len - 1)] joins the
+ * scaled (and capped) score. */
+int spd_attn_general_keys(void* out, const void* q, const void* k_pool, const void* v_pool,
+                          const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
+                          const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                          int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                          int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
+                          float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
+                          int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
+                          int64_t v_slot_stride, int block_size, int block_run_len, int64_t block_base, int keep_first,
+                          const float* dist_bias, int dist_bias_len, int dtype, spd_stream_t stream);
 /* Writes the rows of the blocks that a batch's new tokens complete (their K / V are in the pool already): the mean over
  * the block's token rows of k_pool (rows of k_row_elems) and v_pool (v_row_elems; v_pool NULL: keys only), summed in
  * fp32.  Decode (seq_lens) or ragged extend (max_extend_len: host-side bound of extend_lens); slot 0 is padding. */

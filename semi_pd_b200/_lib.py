@@ -22,6 +22,7 @@ SPD_F16 = 1
 SPD_F32 = 2
 SPD_EPI_NONE = 0
 SPD_EPI_SILU_MUL = 1
+SPD_EPI_GELU = 2
 
 _p = C.c_void_p
 _i64 = C.c_int64
@@ -94,7 +95,7 @@ SIGNATURES = {
     "spd_act_and_mul": (_i, [_p, _p, _i64, _i64, _i, _f, _f, _i, _p]),
     "spd_headnorm_gate": (_i, [_p, _p, _p, _i64, _i, _i, _i64, _f, _p, _i, _i, _i, _p]),
     "spd_linear_simt": (_i, [_p, _p, _p, _i64, _i64, _i64, _i64, _i64, _i64, _p, _i64, _i, _i, _p]),
-    "spd_moe_route_scores": (_i, [_p, _p, _p, _i64, _i64, _i, _i, _i, _i, _f, _p, _i, _i, _p]),
+    "spd_moe_route_scores": (_i, [_p, _p, _p, _i64, _i64, _i, _i, _i, _i, _f, _p, _i, _i, _i, _p]),
     "spd_residual_rmsnorm2": (_i, [_p, _p, _p, _p, _p, _p, _p, _i64, _i64, _f, _f, _i, _p]),
     "spd_linear_simt_block_diag": (_i, [_p, _p, _p, _i64, _i64, _i64, _i64, _i64, _i64, _i, _i64, _i64, _i, _p]),
     "spd_gated_recurrence": (
@@ -110,7 +111,7 @@ SIGNATURES = {
     "spd_head_gate_sigmoid": (_i, [_p, _p, _p, _i64, _i, _i, _i64, _i64, _i, _p]),
     "spd_scale_f32": (_i, [_p, _i64, _f, _p]),
     "spd_moe_gather_scaled": (_i, [_p, _p, _p, _p, _p, _i64, _i, _i64, _i64, _i, _p]),
-    "spd_moe_combine_gated": (_i, [_p, _p, _p, _p, _p, _p, _i64, _i64, _i, _i64, _i, _p]),
+    "spd_moe_combine_gated": (_i, [_p, _p, _p, _p, _p, _p, _i64, _p, _i64, _i64, _i, _i64, _i, _p]),
     "spd_kv_store": (_i, [_p, _p, _p, _p, _p, _i64, _i64, _i64, _i64, _i64, _i, _p]),
     "spd_attn_general": (
         _i,
@@ -146,6 +147,11 @@ SIGNATURES = {
     "spd_heads_gate": (_i, [_p, _p, _p, _p, _i64, _i, _i, _i64, _i64, _i64, _f, _f, _f, _i, _p]),
     "spd_residual_postnorm": (_i, [_p, _p, _p, _p, _p, _i64, _i64, _f, _f, _i, _p]),
     "spd_softcap_f32": (_i, [_p, _i64, _f, _p]),
+    "spd_attn_general_keys": (
+        _i,
+        [_p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i64, _i64, _i, _i, _i, _i, _i64, _i64, _i64, _f, _i, _p, _p,
+         _f, _i, _i64, _f, _i, _i64, _i, _i, _i64, _i, _p, _i, _i, _p],
+    ),
     "spd_attn_general_blocks": (
         _i,
         [_p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i64, _i64, _i, _i, _i, _i, _i64, _i64, _i64, _f, _i, _p, _p,

@@ -68,7 +68,8 @@ class RadixAttention:
                  sliding_window_size: int = -1, is_cross_attention: bool = False, prefix: str = "",
                  sinks: Optional[torch.Tensor] = None, distance_slopes: Optional[torch.Tensor] = None,
                  query_temperature: Optional[tuple] = None, general: bool = False, num_v_heads: int = 0,
-                 v_slot_stride: int = 0, block_pool: int = 0):
+                 v_slot_stride: int = 0, block_pool: int = 0, keep_first: int = 0,
+                 distance_bias: Optional[torch.Tensor] = None):
         self.tp_q_head_num = num_heads
         self.tp_k_head_num = num_kv_heads
         self.tp_v_head_num = num_kv_heads
@@ -96,6 +97,10 @@ class RadixAttention:
         # also the general kernel's: tokens per pooled block; the tokens before the window are seen as one mean key and
         # value per complete block of that many tokens (0: not at all).  Their rows belong to the layer's KV pool.
         self.block_pool = int(block_pool)
+        # also the general kernel's: a sequence's first keep_first tokens stay visible when the window has moved past
+        # them; a bias per head and distance (fp32 [heads, distances], the last entry shared by all further distances)
+        self.keep_first = int(keep_first) if self.sliding_window_size > 0 else 0
+        self.distance_bias = distance_bias
         self.general = bool(general or sinks is not None or distance_slopes is not None or query_temperature
                             or self.sliding_window_size > 0 or self.v_head_dim != self.qk_head_dim)
         self.k_scale = None
@@ -171,14 +176,15 @@ class SpdAttnBackend(AttentionBackend):
         return 1
 
     def _forward_general(self, q, layer: RadixAttention, forward_batch: ForwardBatch):
-        """Window / sink / distance bias / query temperature / k_dim != v_dim / float32: the general
+        """Window (with kept first tokens) / sink / distance bias / query temperature / k_dim != v_dim / float32: the general
         kernel, decode and ragged extend alike, reading the batch's device-side metadata."""
         k_buf, v_buf = forward_batch.token_to_kv_pool.get_kv_buffer(layer.layer_id)
         coef, every = layer.query_temperature or (0.0, 0)
         common = dict(num_q_heads=layer.tp_q_head_num, num_kv_heads=layer.tp_k_head_num, head_dim=layer.qk_head_dim,
                       v_dim=layer.v_head_dim, sm_scale=layer.scaling, window=layer.sliding_window_size,
                       sinks=layer.sinks, slopes=layer.distance_slopes, qtemp_coef=coef, qtemp_every=every,
-                      softcap=layer.logit_cap, num_v_heads=layer.num_v_heads, v_slot_stride=layer.v_slot_stride)
+                      softcap=layer.logit_cap, num_v_heads=layer.num_v_heads, v_slot_stride=layer.v_slot_stride,
+                      keep_first=layer.keep_first, dist_bias=layer.distance_bias)
         r2t = forward_batch.req_to_token_pool.req_to_token
         if layer.block_pool:
             pool = forward_batch.token_to_kv_pool

@@ -349,9 +349,56 @@ def _fudonex_config(path: str, cfg: dict, **overrides) -> ModelConfig:
     return ModelConfig(name=os.path.basename(os.path.normpath(path)) or "fudonex", **kw)
 
 
+def _kuforax_config(path: str, cfg: dict, **overrides) -> ModelConfig:
+    """config.json of the Kuforax family: {"architecture", "vocab", "width", "norm": {"eps"}, "layers": [{"type", "mixer",
+    "mlp"}, ...], "loop": {"start", "stop", "times"}}.  Mixers: "attention" {heads, kv_heads, dim, vdim, scale, mask: {size,
+    keep_first}, rot: {dims, base, scaling: {factor, original, fast, slow}}} (the values are the keys), "attention_2"
+    {heads, kv_heads, dim, vdim, scale, bias_max, mask: {size}}.  Feed-forward: {"kind": "moe", "router": {experts, top,
+    identity, groups: {count, keep}}, "expert": {ff}, "shared": {ff} | null} or null.  `layer_specs` lists the layer RUNS
+    (see expand_loop); every size and constant is carried per layer."""
+    layers = cfg["layers"]
+    for i, spec in enumerate(layers):
+        if spec["type"] not in ("attention", "attention_2"):
+            raise ValueError(f"layer {i}: unknown mixer type {spec['type']!r}")
+        m = spec["mixer"]
+        if int(m["heads"]) % int(m.get("kv_heads", m["heads"])):
+            raise ValueError(f"layer {i}: {m['heads']} heads are not a multiple of {m['kv_heads']} kv heads")
+        mask = m.get("mask") or {}
+        if mask.get("size") is not None and int(mask["size"]) < 1:
+            raise ValueError(f"layer {i}: mask.size {mask['size']} must be positive")
+        if int(mask.get("keep_first") or 0) < 0:
+            raise ValueError(f"layer {i}: mask.keep_first {mask['keep_first']} is negative")
+        if spec["type"] == "attention":
+            rot = int((m.get("rot") or {}).get("dims") or 0)
+            if rot % 2 or rot > int(m["dim"]):
+                raise ValueError(f"layer {i}: rot.dims {rot} must be even and at most dim {m['dim']}")
+            if int(m.get("vdim", m["dim"])) != int(m["dim"]):
+                raise ValueError(f"layer {i}: the values are the keys, so vdim {m['vdim']} must equal dim {m['dim']}")
+        mlp = spec.get("mlp")
+        if mlp is None:
+            continue
+        if mlp.get("kind", "moe") != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        r = mlp["router"]
+        n, groups = int(r["experts"]) + int(r.get("identity") or 0), r.get("groups") or {}
+        count, keep = int(groups.get("count") or 1), int(groups.get("keep") or 1)
+        if n % count or not 1 <= keep <= count or int(r["top"]) > n // count * keep:
+            raise ValueError(f"layer {i}: {n} router outputs in {count} groups, {keep} kept, {r['top']} chosen")
+    runs = expand_loop(layers, cfg.get("loop") or None)
+    kw = dict(model_type="kuforax", hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]),
+              num_hidden_layers=len(runs), rms_norm_eps=float(cfg["norm"]["eps"]), layer_specs=runs,
+              # summary fields other components print or size by; the per-layer values rule
+              num_attention_heads=max(int(s["mixer"]["heads"]) for s in runs),
+              num_key_value_heads=max(int(s["mixer"].get("kv_heads", s["mixer"]["heads"])) for s in runs),
+              head_dim=max(int(s["mixer"]["dim"]) for s in runs), intermediate_size=0,
+              max_position_embeddings=int(cfg.get("context", 8192)))
+    kw.update(overrides)
+    return ModelConfig(name=os.path.basename(os.path.normpath(path)) or "kuforax", **kw)
+
+
 # config.json "architecture" -> reader
 _ARCHITECTURE_READERS = {"Rimidra": _rimidra_config, "Nupovik": _nupovik_config, "Matepel": _matepel_config,
-                         "Sugelix": _sugelix_config, "Fudonex": _fudonex_config}
+                         "Sugelix": _sugelix_config, "Fudonex": _fudonex_config, "Kuforax": _kuforax_config}
 
 
 def load_model_config(path: str, **overrides) -> ModelConfig:

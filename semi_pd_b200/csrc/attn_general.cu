@@ -1,7 +1,7 @@
 // Softmax attention over the paged KV pool with the options the tcgen05 kernels do not have:
-// a sliding window, a learned per-head sink in the denominator, a linear distance bias, a
-// position-dependent query temperature, key size != value size, pooled blocks of the tokens that lie
-// before the window (key_blocks.cuh), and 32-bit storage.  Decode and
+// a sliding window (with the first tokens kept), a learned per-head sink in the denominator, a distance
+// bias (linear, or a table per head), a position-dependent query temperature, key size != value size,
+// pooled blocks of the tokens that lie before the window (key_blocks.cuh), and 32-bit storage.  Decode and
 // ragged extend (chunked prefill, mixed batches) are the same kernel: one warp owns one (query
 // token, query head), walks its visible keys in tiles of 32 (one key per lane for the scores, one
 // slice of the value row per lane for the output) and keeps the online-softmax state in fp32.
@@ -62,7 +62,7 @@ attn_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __res
                     const int32_t* __restrict__ extend_start_loc, int batch, int64_t total_tokens, int H, int G,
                     int dk, int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale,
                     int window, const float* __restrict__ sinks, const float* __restrict__ slopes, float qtemp_coef,
-                    int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
+                    int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db) {
   extern __shared__ float q_smem[];  // [4][dk]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   // item = h * tokens_padded + t with tokens_padded a multiple of 4: the warps of a CTA share a head
@@ -99,6 +99,7 @@ attn_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __res
   __syncwarp();
 
   const float slope = slopes != nullptr ? slopes[h] : 0.f;
+  const float* brow = db.table != nullptr ? db.table + (int64_t)h * db.len : nullptr;
   float m = -INFINITY, l = 0.f;
   if (sinks != nullptr) { m = sinks[h]; l = 1.f; }
   float acc[VMAX];
@@ -116,7 +117,9 @@ attn_general_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __res
       slot = key_row(kb, page, e, nb, j_lo);
       s = dot_row<T>(qs, k_pool + ((int64_t)slot * G + g) * dk, dk);
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-      s -= slope * (float)(n_keys - 1 - e);  // distance of a token (blocks come without a slope)
+      const int64_t dist = key_distance(e, nb, pos, n_keys);
+      s -= slope * (float)dist;
+      if (brow != nullptr) s += distance_bias(brow, db.len, dist);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);  // m = -inf (first tile, no sink): 0
@@ -156,7 +159,7 @@ attn_general_decode_kernel(T* __restrict__ out, const T* __restrict__ q, const T
                            int G, int dk, int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride,
                            float sm_scale, int window, const float* __restrict__ sinks,
                            const float* __restrict__ slopes, float qtemp_coef, int qtemp_every, float softcap, int Gv,
-                           int64_t v_slot, KeyBlocks kb) {
+                           int64_t v_slot, KeyBlocks kb, DistanceBias db) {
   extern __shared__ float dec_smem[];  // q [dk] | m [4] | l [4] | acc [4][dv]
   float* qs = dec_smem;
   float* sm_m = qs + dk;
@@ -174,6 +177,7 @@ attn_general_decode_kernel(T* __restrict__ out, const T* __restrict__ q, const T
   for (int d = threadIdx.x; d < dk; d += 128) qs[d] = to_f32<T>(q[(int64_t)r * q_stride + (int64_t)h * dk + d]) * qmul;
   __syncthreads();
   const float slope = slopes != nullptr ? slopes[h] : 0.f;
+  const float* brow = db.table != nullptr ? db.table + (int64_t)h * db.len : nullptr;
   float m = -INFINITY, l = 0.f;
   float acc[VMAX];
 #pragma unroll
@@ -189,7 +193,9 @@ attn_general_decode_kernel(T* __restrict__ out, const T* __restrict__ q, const T
       slot = key_row(kb, page, e, nb, j_lo);
       s = dot_row<T>(qs, k_pool + ((int64_t)slot * G + g) * dk, dk);
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-      s -= slope * (float)(n_keys - 1 - e);  // distance of a token (blocks come without a slope)
+      const int64_t dist = key_distance(e, nb, pos, n_keys);
+      s -= slope * (float)dist;
+      if (brow != nullptr) s += distance_bias(brow, db.len, dist);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);
@@ -288,7 +294,7 @@ attn_general_decode_group_kernel(T* __restrict__ out, const T* __restrict__ q, c
                                  int H, int G, int dk, int64_t q_stride, int64_t out_stride, int64_t r2t_stride,
                                  float sm_scale, int window, const float* __restrict__ sinks,
                                  const float* __restrict__ slopes, float qtemp_coef, int qtemp_every, int q_bytes,
-                                 float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
+                                 float softcap, int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db) {
   constexpr int N = 16 / (int)sizeof(T);
   constexpr int DV = 32 * VPL;
   constexpr int vstride = DV * (int)sizeof(T) + 16;
@@ -373,14 +379,15 @@ attn_general_decode_group_kernel(T* __restrict__ out, const T* __restrict__ q, c
         }
       }
     }
-    const float dist = (float)(n_keys - 1 - (e0 + lane));
+    const int64_t dist = key_distance(valid ? e0 + lane : n_keys - 1, nb, pos, n_keys);
     float p[RMAX];
 #pragma unroll
     for (int rr = 0; rr < RMAX; ++rr) {
       p[rr] = 0.f;
       if (rr < R) {
         const float sc = softcap > 0.f ? softcap * tanhf(s[rr] / softcap) : s[rr];
-        const float sv = valid ? sc - slope[rr] * dist : -INFINITY;
+        float sv = valid ? sc - slope[rr] * (float)dist : -INFINITY;
+        if (valid && db.table != nullptr) sv += distance_bias(db.table + (int64_t)(g * R + rr) * db.len, db.len, dist);
         const float m_new = fmaxf(m[rr], warp_max(sv));  // finite: the tile has at least one key
         const float corr = expf(m[rr] - m_new);          // first tile (m = -inf): 0
         p[rr] = valid ? expf(sv - m_new) : 0.f;
@@ -447,7 +454,7 @@ int attn_general_decode_group_launch(size_t smem, int q_bytes, int64_t batch, cu
                                      const int64_t* req_pool_indices, const int64_t* seq_lens, int H, int G, int dk,
                                      int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                                      const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every,
-                                     float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
+                                     float softcap, int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db) {
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
     SPD_CUDA(cudaFuncSetAttribute(attn_general_decode_group_kernel<T, VPL, RMAX, NW>,
@@ -457,7 +464,7 @@ int attn_general_decode_group_launch(size_t smem, int q_bytes, int64_t batch, cu
   SPD_CUDA(launch(attn_general_decode_group_kernel<T, VPL, RMAX, NW>, dim3((unsigned)batch, (unsigned)G), dim3(NW * 32), smem,
                   stream, /*pdl=*/false, (T*)out, (const T*)q, (const T*)k_pool, (const T*)v_pool, req_to_token,
                   req_pool_indices, seq_lens, H, G, dk, q_stride, out_stride, r2t_stride, sm_scale, window, sinks, slopes,
-                  qtemp_coef, qtemp_every, q_bytes, softcap, Gv, v_slot, kb));
+                  qtemp_coef, qtemp_every, q_bytes, softcap, Gv, v_slot, kb, db));
   return 0;
 }
 
@@ -557,13 +564,13 @@ int attn_general_mma_try(void* out, const void* q, const void* k_pool, const voi
                          const int32_t* extend_start_loc, int64_t batch, int64_t max_extend_len, int H, int G, int dk,
                          int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                          const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap,
-                         int Gv, int64_t v_slot, KeyBlocks kb, int dtype, cudaStream_t stream);
+                         int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db, int dtype, cudaStream_t stream);
 
 int attn_general_mma_decode_try(void* out, const void* q, const void* k_pool, const void* v_pool,
                                 const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
                                 int64_t batch, int H, int G, int dk, int dv, int64_t q_stride, int64_t out_stride,
                                 int64_t r2t_stride, float sm_scale, int window, const float* sinks, const float* slopes,
-                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb,
+                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db,
                                 int dtype, cudaStream_t stream);
 
 }  // namespace spd
@@ -598,7 +605,7 @@ int spd_pool_key_blocks(void* k_pool, void* v_pool, const int32_t* req_to_token,
   const int64_t rows = seq_lens != nullptr ? 1 : max_extend_len;
   if (batch == 0 || rows <= 0) return 0;
   SPD_REQUIRE(batch <= 65535, SPD_E_SHAPE, "spd_pool_key_blocks: batch too large");
-  const KeyBlocks kb{block_size, block_run_len, (block_run_len + block_size - 1) / block_size, block_base};
+  const KeyBlocks kb{block_size, block_run_len, (block_run_len + block_size - 1) / block_size, block_base, 0};
   const int64_t blocks = (rows + block_size - 1) / block_size;  // n new tokens complete at most that many
   SPD_DISPATCH_ANY(dtype, {
     constexpr int N = 16 / (int)sizeof(T);
@@ -617,15 +624,15 @@ int spd_pool_key_blocks(void* k_pool, void* v_pool, const int32_t* req_to_token,
   return 0;
 }
 
-int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const void* v_pool,
-                            const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
-                            const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
-                            int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
-                            int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
-                            float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
-                            int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
-                            int64_t v_slot_stride, int block_size, int block_run_len,
-                                int64_t block_base, int dtype, spd_stream_t stream) {
+int spd_attn_general_keys(void* out, const void* q, const void* k_pool, const void* v_pool,
+                          const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
+                          const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                          int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                          int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
+                          float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
+                          int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
+                          int64_t v_slot_stride, int block_size, int block_run_len, int64_t block_base, int keep_first,
+                          const float* dist_bias, int dist_bias_len, int dtype, spd_stream_t stream) {
   if (num_v_heads <= 0) num_v_heads = num_kv_heads;
   if (v_slot_stride <= 0) v_slot_stride = (int64_t)num_v_heads * v_dim;
   const int Gv = num_v_heads;
@@ -634,8 +641,13 @@ int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const 
               "spd_attn_general: kv heads %d not a multiple of value heads %d", num_kv_heads, num_v_heads);
   SPD_REQUIRE(block_size == 0 || (block_size > 0 && block_run_len > 0 && block_base > 0 && window > 0 && slopes == nullptr),
               SPD_E_BADARG, "spd_attn_general: pooled blocks need a window, a run length and a base row, and no distance bias");
+  SPD_REQUIRE(keep_first >= 0 && (keep_first == 0 || (window > 0 && block_size == 0)), SPD_E_BADARG,
+              "spd_attn_general: kept first tokens need a window and exclude pooled blocks");
+  SPD_REQUIRE(dist_bias == nullptr || (dist_bias_len > 0 && block_size == 0), SPD_E_BADARG,
+              "spd_attn_general: a distance table needs entries and excludes pooled blocks");
   const KeyBlocks kb{block_size, block_run_len, block_size > 0 ? (block_run_len + block_size - 1) / block_size : 0,
-                     block_base};
+                     block_base, keep_first};
+  const DistanceBias db{dist_bias, dist_bias_len};
   SPD_REQUIRE(out && q && k_pool && v_pool && req_to_token && req_pool_indices, SPD_E_BADARG,
               "spd_attn_general: null pointer");
   SPD_REQUIRE(seq_lens != nullptr || (prefix_lens && extend_lens && extend_start_loc), SPD_E_BADARG,
@@ -653,7 +665,7 @@ int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const 
       const int rc = attn_general_mma_decode_try(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, batch,
                                                  num_q_heads, num_kv_heads, head_dim, v_dim, q_stride, out_stride,
                                                  req_to_token_stride, sm_scale, window, sinks, slopes, qtemp_coef,
-                                                 qtemp_every, softcap, Gv, v_slot, kb, dtype, as_stream(stream));
+                                                 qtemp_every, softcap, Gv, v_slot, kb, db, dtype, as_stream(stream));
       if (rc != 1) return rc;
     }
     // grouped form: 16-byte rows, v_dim 32 x {1, 2, 4, 8}, up to 8 query heads per key/value head
@@ -673,7 +685,7 @@ int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const 
 #define SPD_GRP_ARGS                                                                                                  \
   gsmem, q_bytes, batch, as_stream(stream), out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens,         \
       num_q_heads, num_kv_heads, head_dim, q_stride, out_stride, req_to_token_stride, sm_scale, window, sinks, slopes, \
-      qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb
+      qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, db
 #define SPD_GRP_R(TT, VPL)                                                                     \
   do {                                                                                         \
     if (R <= 1) return nw == 8 ? attn_general_decode_group_launch<TT, VPL, 1, 8>(SPD_GRP_ARGS)  \
@@ -705,7 +717,7 @@ int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const 
                       as_stream(stream), /*pdl=*/false, (T*)out, (const T*)q, (const T*)k_pool, (const T*)v_pool,
                       req_to_token, req_pool_indices, seq_lens, num_q_heads, num_kv_heads, head_dim, v_dim, q_stride,
                       out_stride, req_to_token_stride, sm_scale, window, sinks, slopes, qtemp_coef, qtemp_every, softcap,
-                      Gv, v_slot, kb));
+                      Gv, v_slot, kb, db));
     });
     return 0;
   }
@@ -713,7 +725,7 @@ int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const 
     const int rc = attn_general_mma_try(out, q, k_pool, v_pool, req_to_token, req_pool_indices, prefix_lens, extend_lens,
                                         extend_start_loc, batch, max_extend_len, num_q_heads, num_kv_heads, head_dim,
                                         v_dim, q_stride, out_stride, req_to_token_stride, sm_scale, window, sinks, slopes,
-                                        qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, dtype, as_stream(stream));
+                                        qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, db, dtype, as_stream(stream));
     if (rc != 1) return rc;
   }
   const int64_t tokens4 = (total_tokens + 3) / 4 * 4;
@@ -726,9 +738,25 @@ int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const 
                     (T*)out, (const T*)q, (const T*)k_pool, (const T*)v_pool, req_to_token, req_pool_indices, seq_lens,
                     prefix_lens, extend_lens, extend_start_loc, (int)batch, total_tokens, num_q_heads, num_kv_heads,
                     head_dim, v_dim, q_stride, out_stride, req_to_token_stride, sm_scale, window, sinks, slopes,
-                    qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb));
+                    qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, db));
   });
   return 0;
+}
+
+int spd_attn_general_blocks(void* out, const void* q, const void* k_pool, const void* v_pool,
+                            const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
+                            const int32_t* prefix_lens, const int32_t* extend_lens, const int32_t* extend_start_loc,
+                            int64_t batch, int64_t total_tokens, int num_q_heads, int num_kv_heads, int head_dim,
+                            int v_dim, int64_t q_stride, int64_t out_stride, int64_t req_to_token_stride,
+                            float sm_scale, int window, const float* sinks, const float* slopes, float qtemp_coef,
+                            int qtemp_every, int64_t max_extend_len, float softcap, int num_v_heads,
+                            int64_t v_slot_stride, int block_size, int block_run_len, int64_t block_base, int dtype,
+                            spd_stream_t stream) {
+  return spd_attn_general_keys(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, prefix_lens, extend_lens,
+                               extend_start_loc, batch, total_tokens, num_q_heads, num_kv_heads, head_dim, v_dim, q_stride,
+                               out_stride, req_to_token_stride, sm_scale, window, sinks, slopes, qtemp_coef, qtemp_every,
+                               max_extend_len, softcap, num_v_heads, v_slot_stride, block_size, block_run_len, block_base,
+                               0, nullptr, 0, dtype, stream);
 }
 
 int spd_attn_general_ex(void* out, const void* q, const void* k_pool, const void* v_pool,

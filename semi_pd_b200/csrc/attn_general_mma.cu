@@ -1,10 +1,10 @@
-// Tensor-core prefill path of the general attention (window, sink, distance bias, query temperature,
+// Tensor-core prefill path of the general attention (window, kept first tokens, sink, distance bias, query temperature,
 // key size != value size) for 16-bit models: a CTA owns 64 consecutive query rows of one request and
 // one query head, its four warps 16 rows each; K / V tiles of 64 keys are gathered through the page
 // table with 16-byte cp.async into a double-buffered shared-memory ring, S = Q K^T and O += P V run
 // on warp-level mma.sync.m16n8k16 (fp32 accumulators), and the online softmax — scale, temperature,
 // bias, window mask, sink — is fp32 in the exp2 domain.  Only the keys a tile can see are visited:
-// [first row - window + 1, last row], preceded by the pooled blocks it can see.  The CUDA-core kernel of attn_general.cu keeps decode, float32
+// [first row - window + 1, last row], preceded by the pooled blocks or kept first tokens it can see.  The CUDA-core kernel of attn_general.cu keeps decode, float32
 // models and head sizes outside the instantiated set.  (mma.sync, not tcgen05: the first tensor-core
 // kernel of this mechanism.)
 #include "common.cuh"
@@ -15,6 +15,7 @@
 namespace spd {
 
 constexpr int kGmBQ = 64, kGmBK = 64, kGmThreads = 128;
+constexpr int kGmBiasMax = 4096;  // longest distance table that is kept in shared memory
 constexpr float kLog2e = 1.4426950408889634f;
 
 template <typename T>
@@ -59,7 +60,7 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
                         const int32_t* __restrict__ extend_lens, const int32_t* __restrict__ extend_start_loc, int H,
                         int G, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                         const float* __restrict__ sinks, const float* __restrict__ slopes, float qtemp_coef,
-                        int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
+                        int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db) {
   constexpr int LDK = DK + 8, LDV = DV + 8;  // +16 B per row: ldmatrix rows fall into distinct banks
   extern __shared__ __align__(16) unsigned char gm_smem[];
   T* sQ = reinterpret_cast<T*>(gm_smem);   // [BQ][LDK]
@@ -83,8 +84,9 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
   }
   const int64_t j_hi = i0 + nq - 1;
   const int64_t j_lo = window > 0 ? (i0 - window + 1 > 0 ? i0 - window + 1 : 0) : 0;
-  // the tile's keys in one list: the NB blocks its last row sees, then the tokens j_lo .. j_hi
-  const int NB = (int)key_blocks_seen(kb, j_hi, window), n_keys = NB + (int)(j_hi - j_lo) + 1;
+  // the tile's keys in one list: the NB blocks its last row sees or the NB kept tokens before its first row's window,
+  // then the tokens j_lo .. j_hi
+  const int NB = (int)key_blocks_seen(kb, kb.size > 0 ? j_hi : i0, window), n_keys = NB + (int)(j_hi - j_lo) + 1;
   const int ntiles = (n_keys - 1) / kGmBK + 1;
   // pool rows of a tile's keys (-1 past the end), found two tiles ahead of their use
   __shared__ int slots[2][kGmBK];
@@ -118,13 +120,14 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
 
   const int rl[2] = {warp * 16 + (lane >> 2), warp * 16 + (lane >> 2) + 8};
   const int64_t pi[2] = {i0 + rl[0], i0 + rl[1]};
-  // what a row sees of the list: blocks [0, nbx), tokens [lo, hi] (nothing for rows past the portion)
+  // what a row sees of the list: front entries [0, nbx), tokens [lo, hi] (nothing for rows past the portion).  Kept tokens
+  // are the list's first `keep` entries whether they stand in front of the window or inside it.
   int nbx[2], lo[2], hi[2];
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     const bool ok = pi[x] <= j_hi;
-    nbx[x] = ok ? (int)key_blocks_seen(kb, pi[x], window) : 0;
     hi[x] = ok ? NB + (int)(pi[x] - j_lo) : -1;
+    nbx[x] = !ok ? 0 : kb.size > 0 ? (int)key_blocks_seen(kb, pi[x], window) : (kb.keep <= hi[x] ? kb.keep : hi[x] + 1);
     lo[x] = window > 0 && pi[x] - window + 1 > j_lo ? NB + (int)(pi[x] - window + 1 - j_lo) : NB;
   }
   float sc[2], scc[2];  // score multipliers into the exp2 domain, and (with a cap) into units of the cap
@@ -137,6 +140,14 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
   }
   const float capl = softcap * kLog2e;
   const float sl = (slopes != nullptr ? slopes[h] : 0.f) * kLog2e;
+  // kept tokens in front of the window lie `gap` positions further back than their place in the list says
+  const int gap = kb.size == 0 ? (int)(j_lo - NB) : 0;
+  const float* brow = db.table != nullptr ? db.table + (int64_t)h * db.len : nullptr;
+  float* s_bias = reinterpret_cast<float*>(sV + 2 * kGmBK * LDV);
+  if (brow != nullptr && db.len <= kGmBiasMax) {  // the head's table in shared memory (the first barrier of the loop publishes it)
+    for (int i = tid; i < db.len; i += kGmThreads) s_bias[i] = brow[i];
+    brow = s_bias;
+  }
   const float sink2 = sinks != nullptr ? sinks[h] * kLog2e : -INFINITY;
   float m[2] = {sink2, sink2}, l[2] = {0.f, 0.f};  // l: this thread's share of the row sum
   float o[DV / 8][4];
@@ -175,18 +186,49 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
     }
     const int eb = t * kGmBK;
     float mx[2] = {-INFINITY, -INFINITY};
+    if (brow != nullptr) {
+      // rows x = 0, 1 are eight apart, columns of neighbouring nb too: row 1 of nb has the distance of row 0 of nb - 1
+      float bt[kGmBK / 8 + 1][2];
+      const int d0 = NB + (int)(pi[0] - j_lo) - eb - (lane & 3) * 2;
 #pragma unroll
-    for (int nb = 0; nb < kGmBK / 8; ++nb)
+      for (int i = 0; i <= kGmBK / 8; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int x = e >> 1;
-        const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
-        const bool ok = (idx >= lo[x] && idx <= hi[x]) || idx < nbx[x];
-        const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc[x]) : s[nb][e] * sc[x];
-        const float v = ok ? z - sl * (float)(hi[x] - idx) : -INFINITY;
-        s[nb][e] = v;
-        mx[x] = fmaxf(mx[x], v);
-      }
+        for (int p = 0; p < 2; ++p) {
+          int d = d0 + 8 - 8 * i - p;
+          d = d < 0 ? 0 : (d < db.len ? d : db.len - 1);  // (a negative distance is masked below)
+          bt[i][p] = brow[d];
+        }
+#pragma unroll
+      for (int nb = 0; nb < kGmBK / 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int x = e >> 1;
+          const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
+          float b = bt[nb + 1 - x][e & 1];
+          if (eb < NB && idx < NB && gap > 0) {
+            const int64_t d = pi[x] - idx;
+            b = brow[d < db.len ? d : db.len - 1];
+          }
+          const bool ok = (idx >= lo[x] && idx <= hi[x]) || idx < nbx[x];
+          const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc[x]) : s[nb][e] * sc[x];
+          const float v = ok ? fmaf(b, kLog2e, z) - sl * (float)(hi[x] - idx + (idx < NB ? gap : 0)) : -INFINITY;
+          s[nb][e] = v;
+          mx[x] = fmaxf(mx[x], v);
+        }
+    } else {
+#pragma unroll
+      for (int nb = 0; nb < kGmBK / 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int x = e >> 1;
+          const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
+          const bool ok = (idx >= lo[x] && idx <= hi[x]) || idx < nbx[x];
+          const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc[x]) : s[nb][e] * sc[x];
+          const float v = ok ? z - sl * (float)(hi[x] - idx + (idx < NB ? gap : 0)) : -INFINITY;
+          s[nb][e] = v;
+          mx[x] = fmaxf(mx[x], v);
+        }
+    }
     float ms[2];
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
@@ -250,18 +292,20 @@ static int gm_launch(void* out, const void* q, const void* k_pool, const void* v
                      const int32_t* extend_start_loc, int64_t batch, int64_t max_extend_len, int H, int G,
                      int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                      const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap, int Gv,
-                     int64_t v_slot, KeyBlocks kb, cudaStream_t stream) {
+                     int64_t v_slot, KeyBlocks kb, DistanceBias db, cudaStream_t stream) {
   constexpr size_t smem = sizeof(T) * ((size_t)kGmBQ * (DK + 8) + 2 * kGmBK * (DK + 8) + 2 * kGmBK * (DV + 8));
+  const size_t bias_bytes = db.table != nullptr && db.len <= kGmBiasMax ? sizeof(float) * (size_t)((db.len + 3) / 4 * 4) : 0;
   static bool configured = false;  // per instantiation
   if (!configured) {
-    SPD_CUDA(cudaFuncSetAttribute(attn_general_mma_kernel<T, DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    SPD_CUDA(cudaFuncSetAttribute(attn_general_mma_kernel<T, DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                  (int)(smem + sizeof(float) * kGmBiasMax)));
     configured = true;
   }
   const dim3 grid((unsigned)((max_extend_len + kGmBQ - 1) / kGmBQ), (unsigned)batch, (unsigned)H);
-  SPD_CUDA(launch(attn_general_mma_kernel<T, DK, DV>, grid, dim3(kGmThreads), smem, stream, /*pdl=*/false, (T*)out,
+  SPD_CUDA(launch(attn_general_mma_kernel<T, DK, DV>, grid, dim3(kGmThreads), smem + bias_bytes, stream, /*pdl=*/false, (T*)out,
                   (const T*)q, (const T*)k_pool, (const T*)v_pool, req_to_token, req_pool_indices, prefix_lens,
                   extend_lens, extend_start_loc, H, G, q_stride, out_stride, r2t_stride, sm_scale, window, sinks, slopes,
-                  qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb));
+                  qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, db));
   return 0;
 }
 
@@ -271,7 +315,7 @@ int attn_general_mma_try(void* out, const void* q, const void* k_pool, const voi
                          const int32_t* extend_start_loc, int64_t batch, int64_t max_extend_len, int H, int G, int dk,
                          int dv, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                          const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap,
-                         int Gv, int64_t v_slot, KeyBlocks kb, int dtype, cudaStream_t stream) {
+                         int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db, int dtype, cudaStream_t stream) {
   if (dtype != SPD_BF16 && dtype != SPD_F16) return 1;
   if (v_slot % 8 != 0) return 1;
   if (max_extend_len < 16 || batch > 65535 || H > 65535) return 1;  // short portions: the CUDA-core kernel
@@ -284,11 +328,11 @@ int attn_general_mma_try(void* out, const void* q, const void* k_pool, const voi
       return gm_launch<__nv_bfloat16, DKV, DVV>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, prefix_lens, \
                                                 extend_lens, extend_start_loc, batch, max_extend_len, H, G, q_stride, \
                                                 out_stride, r2t_stride, sm_scale, window, sinks, slopes, qtemp_coef, \
-                                                qtemp_every, softcap, Gv, v_slot, kb, stream);                          \
+                                                qtemp_every, softcap, Gv, v_slot, kb, db, stream);                          \
     return gm_launch<__half, DKV, DVV>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, prefix_lens,        \
                                        extend_lens, extend_start_loc, batch, max_extend_len, H, G, q_stride,        \
                                        out_stride, r2t_stride, sm_scale, window, sinks, slopes, qtemp_coef,         \
-                                       qtemp_every, softcap, Gv, v_slot, kb, stream);                                   \
+                                       qtemp_every, softcap, Gv, v_slot, kb, db, stream);                                   \
   }
   SPD_GM_CASE(32, 32)
   SPD_GM_CASE(64, 64)
@@ -324,7 +368,7 @@ attn_general_mma_decode_kernel(T* __restrict__ out, const T* __restrict__ q, con
                                const int64_t* __restrict__ req_pool_indices, const int64_t* __restrict__ seq_lens,
                                int H, int G, int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale,
                                int window, const float* __restrict__ sinks, const float* __restrict__ slopes,
-                               float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb) {
+                               float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db) {
   constexpr int LDK = DK + 8, LDV = DV + 8;
   constexpr size_t kQBytes = sizeof(T) * 16 * LDK;
   constexpr size_t kWarpBytes = kGdWarpHdr + sizeof(T) * kGdTK * (LDK + LDV);
@@ -359,6 +403,10 @@ attn_general_mma_decode_kernel(T* __restrict__ out, const T* __restrict__ q, con
   float sl[2];
 #pragma unroll
   for (int x = 0; x < 2; ++x) sl[x] = (slopes != nullptr && rr[x] < R) ? slopes[h0 + rr[x]] * kLog2e : 0.f;
+  const float* brow[2];  // the heads' distance tables
+#pragma unroll
+  for (int x = 0; x < 2; ++x)
+    brow[x] = (db.table != nullptr && rr[x] < R) ? db.table + (int64_t)(h0 + rr[x]) * db.len : nullptr;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};  // l: this thread's share of the row sum
   float o[DV / 8][4];
 #pragma unroll
@@ -369,7 +417,7 @@ attn_general_mma_decode_kernel(T* __restrict__ out, const T* __restrict__ q, con
   constexpr int kc = DK / 8, vc = DV / 8;  // 16-byte chunks per row; vc divides 32, kc is at most 32
   const int64_t j_lo = window > 0 ? (pos - window + 1 > 0 ? pos - window + 1 : 0) : 0;
   const int n_split = gridDim.z;  // CTAs of the cluster that share this (request, head)
-  const int64_t nblk = key_blocks_seen(kb, pos, window), n_keys = nblk + pos - j_lo + 1;  // blocks, then tokens
+  const int64_t nblk = key_blocks_seen(kb, pos, window), n_keys = nblk + pos - j_lo + 1;  // front entries, then tokens
   for (int64_t e0 = kGdTK * ((int64_t)blockIdx.z * NW + warp); e0 < n_keys; e0 += (int64_t)kGdTK * NW * n_split) {
     const int n = (int)(n_keys - e0 < kGdTK ? n_keys - e0 : kGdTK);
     __syncwarp();  // the previous tile has been read
@@ -414,7 +462,12 @@ attn_general_mma_decode_kernel(T* __restrict__ out, const T* __restrict__ q, con
         const int x = e >> 1;
         const int col = nb * 8 + (lane & 3) * 2 + (e & 1);
         const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc) : s[nb][e] * sc;
-        const float v = col < n ? z - sl[x] * (float)(n_keys - 1 - (e0 + col)) : -INFINITY;
+        float v = -INFINITY;
+        if (col < n) {
+          const int64_t dist = key_distance(e0 + col, nblk, pos, n_keys);
+          v = z - sl[x] * (float)dist;
+          if (brow[x] != nullptr) v = fmaf(distance_bias(brow[x], db.len, dist), kLog2e, v);
+        }
         s[nb][e] = v;
         mx[x] = fmaxf(mx[x], v);
       }
@@ -552,7 +605,7 @@ static int gd_launch_nw(void* out, const void* q, const void* k_pool, const void
                         const int64_t* req_pool_indices, const int64_t* seq_lens, int64_t batch, int H, int G,
                         int64_t q_stride, int64_t out_stride, int64_t r2t_stride, float sm_scale, int window,
                         const float* sinks, const float* slopes, float qtemp_coef, int qtemp_every, float softcap, int Gv,
-                        int64_t v_slot, KeyBlocks kb, cudaStream_t stream) {
+                        int64_t v_slot, KeyBlocks kb, DistanceBias db, cudaStream_t stream) {
   constexpr size_t tiles = (size_t)NW * (kGdWarpHdr + sizeof(T) * kGdTK * (DK + 8 + DV + 8));
   constexpr size_t merge = sizeof(float) * (NW + 1) * 16 * (DV + 2);  // the warps' triples + the CTA's own
   constexpr size_t smem = sizeof(T) * 16 * (DK + 8) + (tiles > merge ? tiles : merge);
@@ -567,7 +620,7 @@ static int gd_launch_nw(void* out, const void* q, const void* k_pool, const void
   int split = 1;
   const int64_t pairs = batch * G * ((H / G + 15) / 16);
   const int sms = device_sm_count_cached();
-  const int64_t max_split = window > 0 && kb.size == 0 ? (window + kGdTK * NW - 1) / (kGdTK * NW) : 8;
+  const int64_t max_split = window > 0 && kb.size == 0 ? (window + kb.keep + kGdTK * NW - 1) / (kGdTK * NW) : 8;
   while (split * 2 <= 8 && split * 2 <= max_split && pairs * split * 2 <= sms) split *= 2;
   static const bool no_split = getenv("SPD_ATTN_DECODE_NO_SPLIT") != nullptr;
   if (no_split) split = 1;
@@ -586,7 +639,7 @@ static int gd_launch_nw(void* out, const void* q, const void* k_pool, const void
   SPD_CUDA(cudaLaunchKernelEx(&cfg, attn_general_mma_decode_kernel<T, DK, DV, NW>, (T*)out, (const T*)q,
                               (const T*)k_pool, (const T*)v_pool, req_to_token, req_pool_indices, seq_lens, H, G,
                               q_stride, out_stride, r2t_stride, sm_scale, window, sinks, slopes, qtemp_coef,
-                              qtemp_every, softcap, Gv, v_slot, kb));
+                              qtemp_every, softcap, Gv, v_slot, kb, db));
   return 0;
 }
 
@@ -595,31 +648,31 @@ int attn_general_mma_decode_try(void* out, const void* q, const void* k_pool, co
                                 const int32_t* req_to_token, const int64_t* req_pool_indices, const int64_t* seq_lens,
                                 int64_t batch, int H, int G, int dk, int dv, int64_t q_stride, int64_t out_stride,
                                 int64_t r2t_stride, float sm_scale, int window, const float* sinks, const float* slopes,
-                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb,
+                                float qtemp_coef, int qtemp_every, float softcap, int Gv, int64_t v_slot, KeyBlocks kb, DistanceBias db,
                                 int dtype, cudaStream_t stream) {
   if (dtype != SPD_BF16 && dtype != SPD_F16) return 1;
   if (v_slot % 8 != 0) return 1;
   if ((int64_t)G * ((H / G + 15) / 16) > 65535 || batch >= (1ll << 31)) return 1;
   if (q_stride % 8 != 0 || !aligned16(q) || !aligned16(k_pool) || !aligned16(v_pool)) return 1;
   // short windows do not fill eight warps: four warps then leave room for more CTAs per SM
-  const bool wide = window <= 0 || window > 4 * kGdTK || kb.size > 0;
+  const bool wide = window <= 0 || window + kb.keep > 4 * kGdTK || kb.size > 0;
 #define SPD_GD_CASE(DKV, DVV)                                                                                         \
   if (dk == DKV && dv == DVV) {                                                                                       \
     if (dtype == SPD_BF16)                                                                                            \
       return wide ? gd_launch_nw<__nv_bfloat16, DKV, DVV, 8>(out, q, k_pool, v_pool, req_to_token, req_pool_indices,  \
                                                              seq_lens, batch, H, G, q_stride, out_stride, r2t_stride, \
                                                              sm_scale, window, sinks, slopes, qtemp_coef, qtemp_every, \
-                                                             softcap, Gv, v_slot, kb, stream)                                                  \
+                                                             softcap, Gv, v_slot, kb, db, stream)                                                  \
                   : gd_launch_nw<__nv_bfloat16, DKV, DVV, 4>(out, q, k_pool, v_pool, req_to_token, req_pool_indices,  \
                                                              seq_lens, batch, H, G, q_stride, out_stride, r2t_stride, \
                                                              sm_scale, window, sinks, slopes, qtemp_coef, qtemp_every, \
-                                                             softcap, Gv, v_slot, kb, stream);                                                 \
+                                                             softcap, Gv, v_slot, kb, db, stream);                                                 \
     return wide ? gd_launch_nw<__half, DKV, DVV, 8>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, \
                                                     batch, H, G, q_stride, out_stride, r2t_stride, sm_scale, window,  \
-                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, stream)                   \
+                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, db, stream)                   \
                 : gd_launch_nw<__half, DKV, DVV, 4>(out, q, k_pool, v_pool, req_to_token, req_pool_indices, seq_lens, \
                                                     batch, H, G, q_stride, out_stride, r2t_stride, sm_scale, window,  \
-                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, stream);                  \
+                                                    sinks, slopes, qtemp_coef, qtemp_every, softcap, Gv, v_slot, kb, db, stream);                  \
   }
   SPD_GD_CASE(32, 32)
   SPD_GD_CASE(64, 64)

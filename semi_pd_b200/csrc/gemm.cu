@@ -444,7 +444,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUt
         } else {
           tmem_ld_wait();
 #pragma unroll
-          for (int j = 0; j < kChunk; ++j) v[j] = __uint_as_float(r[j]);
+          for (int j = 0; j < kChunk; ++j)
+            v[j] = kEpi == SPD_EPI_GELU ? gelu_f32(to_f32<T>(from_f32<T>(__uint_as_float(r[j])))) : __uint_as_float(r[j]);
         }
         store_chunk(xt, yt, c, v);
       }
@@ -613,8 +614,8 @@ int spd_gemm(void* C, const void* A, const void* W, int64_t M, int64_t N, int64_
   SPD_REQUIRE(M >= 0 && N > 0 && K > 0, SPD_E_BADARG, "spd_gemm: bad sizes M=%lld N=%lld K=%lld",
               (long long)M, (long long)N, (long long)K);
   SPD_REQUIRE(dtype == SPD_BF16 || dtype == SPD_F16, SPD_E_BADARG, "spd_gemm: bad dtype %d", dtype);
-  SPD_REQUIRE(epilogue == SPD_EPI_NONE || epilogue == SPD_EPI_SILU_MUL, SPD_E_BADARG,
-              "spd_gemm: bad epilogue %d", epilogue);
+  SPD_REQUIRE(epilogue == SPD_EPI_NONE || epilogue == SPD_EPI_SILU_MUL || (epilogue == SPD_EPI_GELU && M > 256 && !out_f32),
+              SPD_E_BADARG, "spd_gemm: bad epilogue %d (M %lld)", epilogue, (long long)M);
   SPD_REQUIRE(K % 8 == 0 && N % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0 && ldc % (out_f32 ? 4 : 8) == 0,
               SPD_E_ALIGN, "spd_gemm: K, N and the leading dimensions must be multiples of 8");
   SPD_REQUIRE(aligned16(A) && aligned16(W) && aligned16(C), SPD_E_ALIGN,
@@ -754,6 +755,10 @@ int spd_gemm(void* C, const void* A, const void* W, int64_t M, int64_t N, int64_
     }
     if ((rc = get_tmap(&tx, A, M, K, lda, kBM))) return rc;
     if ((rc = get_tmap(&ty, W, N, K, ldw, BN))) return rc;
+    if (epilogue == SPD_EPI_GELU) {
+      if (use256) SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, 256, false, SPD_EPI_GELU>(tx, ty, p, grid, st); });
+      SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, 128, false, SPD_EPI_GELU>(tx, ty, p, grid, st); });
+    }
     if (use256) {
       SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, 256, false, SPD_EPI_NONE>(tx, ty, p, grid, st); });
     } else {
@@ -771,7 +776,7 @@ int spd_gemm_grouped(void* C, const void* A, const void* W, int64_t M, int64_t N
   SPD_REQUIRE(C && A && W, SPD_E_BADARG, "spd_gemm_grouped: null pointer");
   SPD_REQUIRE(M >= 0 && N > 0 && K > 0 && num_groups > 0, SPD_E_BADARG, "spd_gemm_grouped: bad sizes");
   SPD_REQUIRE(dtype == SPD_BF16 || dtype == SPD_F16, SPD_E_BADARG, "spd_gemm_grouped: bad dtype %d", dtype);
-  SPD_REQUIRE(epilogue == SPD_EPI_NONE || epilogue == SPD_EPI_SILU_MUL, SPD_E_BADARG,
+  SPD_REQUIRE(epilogue == SPD_EPI_NONE || epilogue == SPD_EPI_SILU_MUL || epilogue == SPD_EPI_GELU, SPD_E_BADARG,
               "spd_gemm_grouped: bad epilogue %d", epilogue);
   SPD_REQUIRE(K % 8 == 0 && N % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0 && ldc % 8 == 0 && a_group_stride % 8 == 0,
               SPD_E_ALIGN, "spd_gemm_grouped: K, N, strides and leading dimensions must be multiples of 8");
@@ -825,6 +830,8 @@ int spd_gemm_grouped(void* C, const void* A, const void* W, int64_t M, int64_t N
       p.y_group_rows = N;
       if ((rc = get_tmap(&ty, W, static_cast<uint64_t>(num_groups) * N, K, ldw, BN))) return rc;
     }
+    if (epilogue == SPD_EPI_GELU)
+      SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, BN, false, SPD_EPI_GELU>(tx, ty, p, grid, st); });
     SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, BN, false, SPD_EPI_NONE>(tx, ty, p, grid, st); });
   }
   // cols mode (block diagonal): C[:, g*N:(g+1)*N] = A[:, g*a_group_stride : +K] * W[g*N:(g+1)*N, :K]^T

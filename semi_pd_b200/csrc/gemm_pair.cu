@@ -235,7 +235,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         } else {
           tmem_ld_wait();
 #pragma unroll
-          for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
+          for (int j = 0; j < 32; ++j)
+            v[j] = kEpi == SPD_EPI_GELU ? gelu_f32(to_f32<T>(from_f32<T>(__uint_as_float(r[j])))) : __uint_as_float(r[j]);
         }
         const int64_t n0 = static_cast<int64_t>(yt) * kBNOut + c;
         if (m < p.m_rows) {
@@ -340,6 +341,8 @@ int gemm_pair_try(void* C, const void* A, const void* W, int64_t M, int64_t N, i
   if ((rc = get_tmap(&tw, W, epilogue == SPD_EPI_SILU_MUL ? 2 * N : N, K, ldw, kPgBN / 2))) return rc;
   if (epilogue == SPD_EPI_SILU_MUL) {
     SPD_DISPATCH_DTYPE(dtype, { return launch_pair_gemm<T, SPD_EPI_SILU_MUL>(ta, tw, p, pairs, stream); });
+  } else if (epilogue == SPD_EPI_GELU) {
+    SPD_DISPATCH_DTYPE(dtype, { return launch_pair_gemm<T, SPD_EPI_GELU>(ta, tw, p, pairs, stream); });
   } else {
     SPD_DISPATCH_DTYPE(dtype, { return launch_pair_gemm<T, SPD_EPI_NONE>(ta, tw, p, pairs, stream); });
   }

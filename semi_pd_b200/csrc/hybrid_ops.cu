@@ -221,13 +221,13 @@ constexpr int kRouteMaxTopK = 16;
 constexpr int kRouteMaxGroups = 32;
 
 // scores s = sigmoid(z) or softmax(z); selection runs on the biased score c = s + correction.  With groups the
-// experts are cut into equal runs of neighbours, every run is ranked by its top-2 biased scores added together,
-// and experts outside the keep_groups highest-ranked runs are ineligible (c = -inf there).  The weight of a
+// experts are cut into equal runs of neighbours, every run is ranked by its largest biased score or (group_top 2)
+// its two largest added together, and experts outside the keep_groups highest-ranked runs are ineligible (c = -inf there).  The weight of a
 // selected expert is its unbiased s (optionally renormalised).
 __global__ void __launch_bounds__(128)
 moe_route_scores_kernel(int32_t* __restrict__ topk_ids, float* __restrict__ topk_w, const float* __restrict__ logits,
                         int64_t ld, int64_t tokens, int E, int k, int score_func, int renorm, float scale,
-                        const float* __restrict__ correction, int num_groups, int keep_groups) {
+                        const float* __restrict__ correction, int num_groups, int keep_groups, int group_top) {
   griddep_wait();
   griddep_launch_dependents();
   const int lane = threadIdx.x & 31;
@@ -286,7 +286,7 @@ moe_route_scores_kernel(int32_t* __restrict__ topk_ids, float* __restrict__ topk
         a1 = hi;
         a2 = lo;
       }
-      if (lane == g) gscore = a1 + (per >= 2 ? a2 : 0.f);
+      if (lane == g) gscore = a1 + (group_top >= 2 && per >= 2 ? a2 : 0.f);
     }
     unsigned kept = 0u;
     for (int j = 0; j < keep_groups; ++j) {
@@ -391,21 +391,30 @@ template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
 moe_combine_gated_kernel(T* __restrict__ out, const T* __restrict__ y, const int32_t* __restrict__ inv_pos,
                          const float* __restrict__ topk_w, const T* __restrict__ shared,
-                         const float* __restrict__ shared_gate, int64_t gate_stride, int top_k, int64_t dim) {
+                         const float* __restrict__ shared_gate, int64_t gate_stride, const T* __restrict__ input,
+                         int64_t input_stride, int top_k, int64_t dim) {
   griddep_wait();
   griddep_launch_dependents();
   const int64_t t = blockIdx.x;
   const float sg = shared_gate != nullptr ? sigmoid_precise(shared_gate[t * gate_stride]) : 1.f;
   constexpr int N = Vec16<T>::kN;
-  if (dim % N == 0 && ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(y) |
-                        reinterpret_cast<uintptr_t>(shared)) & 15u) == 0) {
+  // the row that entry j contributes: an expert's output, or the token's own input row where no expert has it
+  auto row_of = [&](int j) -> const T* {
+    const int64_t r = inv_pos[t * top_k + j];
+    return r >= 0 ? y + r * dim : input != nullptr ? input + t * input_stride : nullptr;
+  };
+  if (dim % N == 0 && input_stride % N == 0 &&
+      ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(shared) |
+        reinterpret_cast<uintptr_t>(input)) & 15u) == 0) {
     for (int64_t i = threadIdx.x * N; i < dim; i += kRowThreads * N) {
       float acc[N];
 #pragma unroll
       for (int k = 0; k < N; ++k) acc[k] = 0.f;
       for (int j = 0; j < top_k; ++j) {
         const float w = topk_w != nullptr ? topk_w[t * top_k + j] : 1.f;
-        const Vec16<T> v = ldv(y + (int64_t)inv_pos[t * top_k + j] * dim + i);
+        const T* row = row_of(j);
+        if (row == nullptr) continue;
+        const Vec16<T> v = ldv(row + i);
 #pragma unroll
         for (int k = 0; k < N; ++k) acc[k] += w * to_f32<T>(v.e()[k]);
       }
@@ -425,7 +434,8 @@ moe_combine_gated_kernel(T* __restrict__ out, const T* __restrict__ y, const int
     float acc = 0.f;
     for (int j = 0; j < top_k; ++j) {
       const float w = topk_w != nullptr ? topk_w[t * top_k + j] : 1.f;
-      acc += w * to_f32<T>(y[(int64_t)inv_pos[t * top_k + j] * dim + i]);
+      const T* row = row_of(j);
+      if (row != nullptr) acc += w * to_f32<T>(row[i]);
     }
     if (shared != nullptr) acc += sg * to_f32<T>(shared[t * dim + i]);
     out[t * dim + i] = from_f32<T>(acc);
@@ -559,12 +569,13 @@ int spd_linear_simt_block_diag(void* C, const void* A, const void* W, int64_t M,
 
 int spd_moe_route_scores(int32_t* topk_ids, float* topk_w, const float* logits, int64_t ld, int64_t tokens,
                          int num_experts, int top_k, int score_func, int renormalize, float scale,
-                         const float* correction, int num_groups, int keep_groups, spd_stream_t stream) {
+                         const float* correction, int num_groups, int keep_groups, int group_top, spd_stream_t stream) {
   SPD_REQUIRE(topk_ids && topk_w && logits, SPD_E_BADARG, "spd_moe_route_scores: null pointer");
   SPD_REQUIRE(num_experts > 0 && num_experts <= kRouteMaxExperts && top_k > 0 && top_k <= kRouteMaxTopK &&
                   top_k <= num_experts && ld >= num_experts && (score_func == 0 || score_func == 1),
               SPD_E_SHAPE, "spd_moe_route_scores: experts %d (max %d), top_k %d (max %d)", num_experts,
               kRouteMaxExperts, top_k, kRouteMaxTopK);
+  SPD_REQUIRE(group_top == 1 || group_top == 2, SPD_E_BADARG, "spd_moe_route_scores: group_top is 1 or 2");
   SPD_REQUIRE(num_groups <= 1 || (num_groups <= kRouteMaxGroups && num_experts % num_groups == 0 && keep_groups >= 1 &&
                                   keep_groups <= num_groups && (int64_t)keep_groups * (num_experts / num_groups) >= top_k),
               SPD_E_SHAPE, "spd_moe_route_scores: %d groups (max %d, dividing the experts), keep %d", num_groups,
@@ -572,7 +583,7 @@ int spd_moe_route_scores(int32_t* topk_ids, float* topk_w, const float* logits, 
   if (tokens == 0) return 0;
   SPD_CUDA(launch(moe_route_scores_kernel, dim3((unsigned)((tokens + 3) / 4)), dim3(128), 0, as_stream(stream),
                   pdl_enabled(), topk_ids, topk_w, logits, ld, tokens, num_experts, top_k, score_func, renormalize,
-                  scale, correction, num_groups, keep_groups));
+                  scale, correction, num_groups, keep_groups, group_top));
   return 0;
 }
 
@@ -589,14 +600,15 @@ int spd_moe_gather_scaled(void* xs, const void* x, const int32_t* row_token, con
 }
 
 int spd_moe_combine_gated(void* out, const void* y, const int32_t* inv_pos, const float* topk_w,
-                          const void* shared, const float* shared_gate, int64_t gate_stride, int64_t tokens,
-                          int top_k, int64_t dim, int dtype, spd_stream_t stream) {
+                          const void* shared, const float* shared_gate, int64_t gate_stride, const void* input,
+                          int64_t input_stride, int64_t tokens, int top_k, int64_t dim, int dtype,
+                          spd_stream_t stream) {
   SPD_REQUIRE(out && y && inv_pos, SPD_E_BADARG, "spd_moe_combine_gated: null pointer");
   if (tokens == 0) return 0;
   SPD_DISPATCH_ANY(dtype, {
     SPD_CUDA(launch(moe_combine_gated_kernel<T>, dim3((unsigned)tokens), dim3(kRowThreads), 0, as_stream(stream),
                     pdl_enabled(), (T*)out, (const T*)y, inv_pos, topk_w, (const T*)shared, shared_gate, gate_stride,
-                    top_k, dim));
+                    (const T*)input, input_stride, top_k, dim));
   });
   return 0;
 }

@@ -55,6 +55,7 @@ __device__ __forceinline__ float act_apply(float z, int act) {
     case 1: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));   // gelu (tanh form)
     case 2: { const float r = fmaxf(z, 0.f); return r * r; }                                        // relu squared
     case 3: return tanhf(z);
+    case 5: return gelu_f32(z);                                                                    // gelu (erf form)
     default: return fmaxf(z, 0.f);                                                                  // relu
   }
 }
@@ -246,7 +247,7 @@ int spd_cast_concat(void* out, const float* a, const float* b, int64_t rows, int
 int spd_activation(void* out, const void* x, int64_t rows, int64_t cols, int64_t x_stride, int act, int dtype,
                    spd_stream_t stream) {
   SPD_REQUIRE(out && x, SPD_E_BADARG, "spd_activation: null pointer");
-  SPD_REQUIRE(rows >= 0 && cols > 0 && x_stride >= cols && act >= 0 && act <= 4, SPD_E_BADARG,
+  SPD_REQUIRE(rows >= 0 && cols > 0 && x_stride >= cols && act >= 0 && act <= 5, SPD_E_BADARG,
               "spd_activation: bad arguments");
   if (rows == 0) return 0;
   SPD_DISPATCH_ANY(dtype, {

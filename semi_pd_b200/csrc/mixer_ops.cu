@@ -4,7 +4,7 @@
 //     block adds in front of its first layer),
 //   * rotary positions over strided "segments" (q, k, v of a merged projection, or the rotated slice of a
 //     latent attention's queries and keys), in the paired or the half-split layout, with the biases of the
-//     projections added first, an RMS norm per head (with or without a weight) where a segment asks for one,
+//     projections added first, an RMS norm per head or over all heads of a row where a segment asks for one,
 //     and the cache write fused,
 //   * the fp32 residual update of layers that norm a sublayer's OUTPUT,
 //   * the step between an attention and its output projection: an elementwise sigmoid gate, optionally on
@@ -110,8 +110,8 @@ struct RotarySegment {
   void* dst;          // head h of token t goes to dst + (to_pool ? loc[t] : t) * dst_row + h * dst_head
   int64_t src_row, dst_row;
   int32_t heads, head_dim, rot, src_head, dst_head, to_pool;
-  const float* norm_w;  // [head_dim] or null (plain unit RMS); read when norm != 0
-  int32_t norm;         // RMS norm over the head's channels, after the bias and before the rotation
+  const float* norm_w;  // [head_dim] (norm 2: [heads * head_dim]) or null (plain unit RMS); read when norm != 0
+  int32_t norm;         // RMS norm after the bias and before the rotation: 1 over the head's channels, 2 over all heads
   float norm_eps;
 };
 struct RotarySegments {
@@ -388,6 +388,113 @@ rotary_segments_norm_kernel(RotarySegments segs, const int64_t* __restrict__ pos
   }
 }
 
+// The form with norms over all heads of a row (norm 2; norm 0 segments beside them): one CTA per token sums the squares
+// of every normed segment, then each work item — VEC channels of a head, in the rotated part together with their
+// partners — is read again (from L1), scaled, rotated and written.  VEC > 1: head_dim, rot / 2 (rot in the paired
+// layout), head and row strides multiples of VEC, 16-byte aligned pointers.
+constexpr int kRowNormThreads = 256;
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowNormThreads)
+rotary_segments_rownorm_kernel(RotarySegments segs, const int64_t* __restrict__ positions,
+                               const int64_t* __restrict__ loc, const float* __restrict__ cos_sin, int rot_max,
+                               int64_t max_positions, int paired) {
+  griddep_wait();
+  griddep_launch_dependents();
+  using V = RotVec<T, VEC>;
+  __shared__ float red[4][kRowNormThreads / 32];
+  const int64_t t = blockIdx.x;
+  int64_t p = positions[t];
+  p = p < 0 ? 0 : (p < max_positions ? p : max_positions - 1);
+  const float* cs = cos_sin != nullptr ? cos_sin + p * rot_max : nullptr;
+  const int half_max = rot_max >> 1;
+  const int64_t slot = loc != nullptr ? loc[t] : 0;
+  float ss[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int sidx = 0; sidx < 4; ++sidx) {
+    if (sidx >= segs.n || segs.seg[sidx].norm != 2) continue;
+    const RotarySegment& sg = segs.seg[sidx];
+    const T* src = reinterpret_cast<const T*>(sg.src) + t * sg.src_row;
+    const int per_head = sg.head_dim / VEC;
+    for (int item = threadIdx.x; item < sg.heads * per_head; item += kRowNormThreads) {
+      const int h = item / per_head, d0 = (item - h * per_head) * VEC;
+      const V v = *reinterpret_cast<const V*>(src + h * sg.src_head + d0);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        const float x = to_f32<T>(v.e[i]) + (sg.bias != nullptr ? sg.bias[h * sg.head_dim + d0 + i] : 0.f);
+        ss[sidx] = fmaf(x, x, ss[sidx]);
+      }
+    }
+    ss[sidx] = warp_sum(ss[sidx]);
+    if ((threadIdx.x & 31) == 0) red[sidx][threadIdx.x >> 5] = ss[sidx];
+  }
+  __syncthreads();
+  for (int sidx = 0; sidx < segs.n; ++sidx) {
+    const RotarySegment& sg = segs.seg[sidx];
+    const T* src = reinterpret_cast<const T*>(sg.src) + t * sg.src_row;
+    T* dst = reinterpret_cast<T*>(sg.dst) + (sg.to_pool ? slot : t) * sg.dst_row;
+    float inv = 1.f;
+    if (sg.norm == 2) {
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < kRowNormThreads / 32; ++i) sum += red[sidx][i];
+      inv = 1.0f / sqrtf(sum / (float)(sg.heads * sg.head_dim) + sg.norm_eps);
+    }
+    const float* nw = sg.norm == 2 ? sg.norm_w : nullptr;
+    const int half = sg.rot >> 1, per_head = sg.head_dim / VEC;
+    for (int item = threadIdx.x; item < sg.heads * per_head; item += kRowNormThreads) {
+      const int h = item / per_head, d0 = (item - h * per_head) * VEC;
+      const T* sp = src + h * sg.src_head;
+      T* dp = dst + h * sg.dst_head;
+      auto read = [&](int d, float (&x)[VEC]) {
+        const V v = *reinterpret_cast<const V*>(sp + d);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          const int c = h * sg.head_dim + d + i;
+          x[i] = (to_f32<T>(v.e[i]) + (sg.bias != nullptr ? sg.bias[c] : 0.f)) * inv * (nw != nullptr ? nw[c] : 1.f);
+        }
+      };
+      auto write = [&](int d, const float (&x)[VEC]) {
+        V v;
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v.e[i] = from_f32<T>(x[i]);
+        *reinterpret_cast<V*>(dp + d) = v;
+      };
+      float a[VEC];
+      if (d0 >= sg.rot) {
+        read(d0, a);
+        write(d0, a);
+      } else if (VEC > 1 && paired) {
+        read(d0, a);
+#pragma unroll
+        for (int i = 0; i + 1 < VEC; i += 2) {
+          const float c = cs[(d0 + i) >> 1], sn = cs[half_max + ((d0 + i) >> 1)];
+          const float x = a[i], y = a[i + 1];
+          a[i] = x * c - y * sn;
+          a[i + 1] = y * c + x * sn;
+        }
+        write(d0, a);
+      } else {
+        // the item of the pair's first channel turns both
+        const int partner = paired ? d0 + 1 : d0 + half;
+        if (paired ? (d0 & 1) != 0 : d0 >= half) continue;
+        float b[VEC];
+        read(d0, a);
+        read(partner, b);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          const int f = paired ? d0 >> 1 : d0 + i;
+          const float c = cs[f], sn = cs[half_max + f];
+          const float x = a[i], y = b[i];
+          a[i] = x * c - y * sn;
+          b[i] = y * c + x * sn;
+        }
+        write(d0, a);
+        write(partner, b);
+      }
+    }
+  }
+}
+
 // The residual update of a layer that norms its sublayer's output: x[row] += y / rms(y) * coef (y null: no update),
 // then out = x in T, or (w given) x / rms(x) * (off + w).  One CTA per row; a row of up to NV vectors per thread stays
 // in registers (VEC = 1: any size, read twice).
@@ -634,6 +741,28 @@ int spd_rotary_segments(const spd_rotary_segment_t* segments, int num_segments, 
                                 s.dst_head, s.to_pool, s.norm_w, s.norm, s.norm_eps};
   }
   if (tokens == 0) return 0;
+  bool row_norm = false, head_norm = false;
+  for (int i = 0; i < num_segments; ++i) {
+    row_norm = row_norm || segs.seg[i].norm == 2;
+    head_norm = head_norm || segs.seg[i].norm == 1;
+    SPD_REQUIRE(segs.seg[i].norm >= 0 && segs.seg[i].norm <= 2, SPD_E_BADARG, "spd_rotary_segments: norm is 0, 1 or 2");
+  }
+  const int vecn = dtype == SPD_F32 ? 4 : 8;
+  bool vec = true;
+  for (int i = 0; i < num_segments; ++i) {
+    const RotarySegment& s = segs.seg[i];
+    vec = vec && s.head_dim % vecn == 0 && (paired ? s.rot : s.rot / 2) % vecn == 0 && s.src_head % vecn == 0 &&
+          s.dst_head % vecn == 0 && s.src_row % vecn == 0 && s.dst_row % vecn == 0 && aligned16(s.src) && aligned16(s.dst);
+  }
+  if (row_norm) {
+    SPD_REQUIRE(!head_norm, SPD_E_BADARG, "spd_rotary_segments: norms per head and per row in one launch");
+    SPD_DISPATCH_ANY(dtype, {
+      auto kern = vec ? rotary_segments_rownorm_kernel<T, 16 / (int)sizeof(T)> : rotary_segments_rownorm_kernel<T, 1>;
+      SPD_CUDA(launch(kern, dim3((unsigned)tokens), dim3(kRowNormThreads), 0, as_stream(stream), pdl_enabled(), segs,
+                      positions, loc, cos_sin, rot_max, max_positions, paired));
+    });
+    return 0;
+  }
   int dim_max = 0, step = 4;  // form with norms: the widest step every segment's sizes allow
   bool any_norm = false;
   for (int i = 0; i < num_segments; ++i) {
@@ -678,13 +807,6 @@ int spd_rotary_segments(const spd_rotary_segment_t* segments, int num_segments, 
                       pdl_enabled(), segs, positions, loc, cos_sin, rot_max, max_positions, paired, pad));
     });
     return 0;
-  }
-  const int vecn = dtype == SPD_F32 ? 4 : 8;
-  bool vec = true;
-  for (int i = 0; i < num_segments; ++i) {
-    const RotarySegment& s = segs.seg[i];
-    vec = vec && s.head_dim % vecn == 0 && (paired ? s.rot : s.rot / 2) % vecn == 0 && s.src_head % vecn == 0 &&
-          s.dst_head % vecn == 0 && s.src_row % vecn == 0 && s.dst_row % vecn == 0 && aligned16(s.src) && aligned16(s.dst);
   }
   SPD_DISPATCH_ANY(dtype, {
     auto kern = vec ? rotary_segments_vec_kernel<T> : rotary_segments_kernel<T>;

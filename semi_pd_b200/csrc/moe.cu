@@ -91,7 +91,7 @@ moe_route_kernel(int32_t* __restrict__ topk_ids, float* __restrict__ topk_w, con
 
 // Single CTA: rows sorted by expert, every expert's rows padded to whole 128-row tiles.
 //   row_token[r]  token feeding sorted row r (-1 = padding row)
-//   inv_pos[i]    sorted row of routing entry i = token * k + j
+//   inv_pos[i]    sorted row of routing entry i = token * k + j (-1: a choice outside the E experts, which owns no row)
 //   tile_group[x] expert of 128-row tile x (-1 = unused tile)
 __global__ void __launch_bounds__(1024)
 moe_align_kernel(int32_t* __restrict__ row_token, int32_t* __restrict__ inv_pos, int32_t* __restrict__ tile_group,
@@ -106,7 +106,8 @@ moe_align_kernel(int32_t* __restrict__ row_token, int32_t* __restrict__ inv_pos,
   const int64_t max_tiles = max_rows / kMoeTile;
   for (int64_t x = tid; x < max_tiles; x += 1024) tile_group[x] = -1;
   __syncthreads();
-  for (int64_t i = tid; i < entries; i += 1024) atomicAdd(&cnt[topk_ids[i]], 1);
+  for (int64_t i = tid; i < entries; i += 1024)
+    if (topk_ids[i] < E) atomicAdd(&cnt[topk_ids[i]], 1);
   __syncthreads();
   if (tid == 0) {
     int o = 0;
@@ -121,6 +122,10 @@ moe_align_kernel(int32_t* __restrict__ row_token, int32_t* __restrict__ inv_pos,
     for (int x = off[e] / kMoeTile; x < off[e + 1] / kMoeTile; ++x) tile_group[x] = e;
   for (int64_t i = tid; i < entries; i += 1024) {
     const int e = topk_ids[i];
+    if (e >= E) {
+      inv_pos[i] = -1;
+      continue;
+    }
     const int pos = off[e] + atomicAdd(&cur[e], 1);
     inv_pos[i] = pos;
     row_token[pos] = static_cast<int32_t>(i / k);

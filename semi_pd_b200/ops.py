@@ -14,7 +14,7 @@ from typing import Optional
 import torch
 
 from . import _lib
-from ._lib import SPD_EPI_NONE, SPD_EPI_SILU_MUL, check, lib
+from ._lib import SPD_EPI_GELU, SPD_EPI_NONE, SPD_EPI_SILU_MUL, check, lib
 
 _DTYPE = {torch.bfloat16: _lib.SPD_BF16, torch.float16: _lib.SPD_F16}
 # the 32-bit capable operators (hybrid model family) additionally take float32
@@ -378,7 +378,8 @@ def moe_route(logits: torch.Tensor, top_k: int, scale: float = 1.0, renormalize:
 
 
 def moe_align(topk_ids: torch.Tensor, num_experts: int):
-    """→ (row_token [R], inv_pos [T*k], tile_group [R/128]) with R = spd_moe_align_rows()."""
+    """→ (row_token [R], inv_pos [T*k], tile_group [R/128]) with R = spd_moe_align_rows().  Choices >= num_experts own
+    no row (inv_pos −1)."""
     _cuda(topk_ids)
     T, k = topk_ids.shape
     R = lib.spd_moe_align_rows(T, k, num_experts)
@@ -631,20 +632,22 @@ def linear_any(x: torch.Tensor, weight: torch.Tensor, out_f32: bool = False) -> 
 
 
 def linear_grouped_any(x_sorted: torch.Tensor, weight: torch.Tensor, tile_group: torch.Tensor, num_groups: int,
-                       n: int, silu_mul: bool = False) -> torch.Tensor:
+                       n: int, silu_mul: bool = False, gelu: bool = False) -> torch.Tensor:
     """Expert-grouped F.linear over 128-row tiles; weight = the experts' [n, K] matrices stacked.
     silu_mul: each expert's block is [gate; up] (2n rows) and the result is silu(gate) * up [rows, n] —
     the tensor-core GEMM applies it to its fp32 accumulators in the epilogue, the CUDA-core route runs
-    the activation kernel on the product."""
+    the activation kernel on the product.  gelu: the erf-form GELU of the product, by the same routes."""
     if (_tc_gemm_ok(x_sorted, weight, n) and x_sorted.shape[1] % 64 == 0
             and os.environ.get("SPD_HYBRID_GEMM", "tc") == "tc"):
         if silu_mul and os.environ.get("SPD_HYBRID_FUSED_ACT", "1") != "1":
             return act_and_mul(linear_grouped_rows(x_sorted, weight, tile_group, num_groups, 2 * n), "silu")
+        if gelu and os.environ.get("SPD_HYBRID_FUSED_ACT", "1") != "1":
+            return activation(linear_grouped_rows(x_sorted, weight, tile_group, num_groups, n), "gelu")
         return linear_grouped_rows(x_sorted, weight, tile_group, num_groups, n,
-                                   epilogue=SPD_EPI_SILU_MUL if silu_mul else SPD_EPI_NONE)
+                                   epilogue=SPD_EPI_SILU_MUL if silu_mul else SPD_EPI_GELU if gelu else SPD_EPI_NONE)
     rows = 2 * n if silu_mul else n
     y = linear_simt(x_sorted, weight, tile_group=tile_group, group_rows=rows, n=rows)
-    return act_and_mul(y, "silu") if silu_mul else y
+    return act_and_mul(y, "silu") if silu_mul else activation(y, "gelu") if gelu else y
 
 
 def linear_silu_mul_any(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
@@ -658,13 +661,22 @@ def linear_silu_mul_any(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     return act_and_mul(linear_any(x, weight), "silu")
 
 
+def linear_gelu_any(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """gelu(x Wᵀ), erf form: in the epilogue of one tensor-core GEMM for prefill-sized 16-bit batches, GEMM + activation
+    kernel otherwise."""
+    if (x.shape[0] >= 257 and _tc_gemm_ok(x, weight, weight.shape[0]) and os.environ.get("SPD_HYBRID_GEMM", "tc") == "tc"
+            and os.environ.get("SPD_HYBRID_FUSED_ACT", "1") == "1"):
+        return linear(x, weight, epilogue=SPD_EPI_GELU)
+    return activation(linear_any(x, weight), "gelu")
+
+
 def moe_route_scores(logits: torch.Tensor, num_experts: int, top_k: int, score_func: str = "sigmoid",
                      renormalize: bool = False, scale: float = 1.0, correction: Optional[torch.Tensor] = None,
-                     num_groups: int = 1, keep_groups: int = 1):
+                     num_groups: int = 1, keep_groups: int = 1, group_top: int = 2):
     """fp32 logits [T, >= E] (row stride free) → (topk_ids int32 [T, k], topk_weights fp32 [T, k]).
     correction (fp32 [E]) biases the selection, never the weights; with num_groups > 1 the experts are cut into
-    equal runs, each run is ranked by its top-2 biased scores added together, and selection is restricted to the
-    keep_groups highest-ranked runs."""
+    equal runs, each run is ranked by its largest biased score (group_top 1) or its two largest added together (2), and
+    selection is restricted to the keep_groups highest-ranked runs."""
     _cuda(logits, correction)
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != num_experts):
         raise RuntimeError("moe_route_scores: correction is fp32 [experts]")
@@ -675,7 +687,8 @@ def moe_route_scores(logits: torch.Tensor, num_experts: int, top_k: int, score_f
     w = torch.empty((T, top_k), device=logits.device, dtype=torch.float32)
     check(lib.spd_moe_route_scores(ids.data_ptr(), w.data_ptr(), logits.data_ptr(), logits.stride(0), T, num_experts,
                                    top_k, {"softmax": 0, "sigmoid": 1}[score_func], 1 if renormalize else 0,
-                                   float(scale), _ptr(correction), int(num_groups), int(keep_groups), _stream()),
+                                   float(scale), _ptr(correction), int(num_groups), int(keep_groups), int(group_top),
+                                   _stream()),
           "spd_moe_route_scores")
     return ids, w
 
@@ -694,16 +707,22 @@ def moe_gather_scaled(x: torch.Tensor, row_token: torch.Tensor, inv_pos: torch.T
 
 def moe_combine_gated(y: torch.Tensor, inv_pos: torch.Tensor, tokens: int, top_k: int,
                       topk_w: Optional[torch.Tensor] = None, shared: Optional[torch.Tensor] = None,
-                      shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      shared_gate: Optional[torch.Tensor] = None,
+                      identity: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Σ_j [w_j] y[row(t, j)] + [sigmoid(shared_gate[t])] shared[t]; shared_gate is an fp32 column
-    (any row stride)."""
-    _cuda(y, inv_pos, topk_w, shared, shared_gate)
+    (any row stride).  identity [tokens, dim] (contiguous rows): what an entry without a row (moe_align: a choice
+    outside the experts) contributes — the experts' input for experts that hand it on; None: nothing."""
+    _cuda(y, inv_pos, topk_w, shared, shared_gate, identity)
+    if identity is not None and (identity.dtype != y.dtype or identity.stride(1) != 1 or identity.shape[1] != y.shape[1]):
+        raise RuntimeError("moe_combine_gated: identity is [tokens, dim] in y's dtype")
     out = torch.empty((tokens, y.shape[1]), device=y.device, dtype=y.dtype)
     gs = shared_gate.stride(0) if shared_gate is not None else 0
     if shared_gate is not None and shared_gate.dtype != torch.float32:
         raise RuntimeError("moe_combine_gated: the shared gate logits are fp32")
     check(lib.spd_moe_combine_gated(out.data_ptr(), y.data_ptr(), inv_pos.data_ptr(), _ptr(topk_w), _ptr(shared),
-                                    _ptr(shared_gate), gs, tokens, top_k, y.shape[1], _dta(y), _stream()),
+                                    _ptr(shared_gate), gs, _ptr(identity),
+                                    identity.stride(0) if identity is not None else 0, tokens, top_k, y.shape[1],
+                                    _dta(y), _stream()),
           "spd_moe_combine_gated")
     return out
 
@@ -832,11 +851,11 @@ def cast_concat(a: torch.Tensor, b: torch.Tensor, dtype: torch.dtype) -> torch.T
     return out
 
 
-_ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "tanh": 3, "relu": 4}
+_ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "tanh": 3, "relu": 4, "gelu": 5}
 
 
 def activation(x: torch.Tensor, act: str) -> torch.Tensor:
-    """act(x) elementwise (silu, gelu_tanh, relu2 = relu squared, tanh, relu); x [rows, cols] with contiguous rows."""
+    """act(x) elementwise (silu, gelu_tanh, relu2 = relu squared, tanh, relu, gelu = the erf form); x [rows, cols] with contiguous rows."""
     _cuda(x)
     if x.dim() != 2 or x.stride(1) != 1:
         raise RuntimeError("activation: x must be [rows, cols] with contiguous rows")
@@ -912,15 +931,21 @@ def attn_general(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, re
                  sinks: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None, qtemp_coef: float = 0.0,
                  qtemp_every: int = 0, seq_lens=None, prefix_lens=None, extend_lens=None, extend_start_loc=None,
                  max_extend_len: int = 0, softcap: float = 0.0, num_v_heads: int = 0,
-                 v_slot_stride: int = 0, blocks: Optional[tuple] = None) -> torch.Tensor:
+                 v_slot_stride: int = 0, blocks: Optional[tuple] = None, keep_first: int = 0,
+                 dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Windowed / sink / distance-biased softmax attention over the paged pool; decode (seq_lens) or
     ragged extend (prefix_lens, extend_lens, extend_start_loc).  q [T, H·head_dim] → [T, H·v_dim].
     max_extend_len > 0 (a host-side bound of extend_lens) lets 16-bit prefill run on the tensor cores.
     softcap > 0 caps the scaled scores by softcap · tanh(· / softcap); num_v_heads < num_kv_heads: key head g
     reads value head g mod num_v_heads; v_slot_stride: elements between two slots of v_pool (values that are
     the first v_dim columns of wider rows).  blocks (size, run_len, base): besides its window a query sees one pooled key
-    and value per block of `size` tokens that lies wholly before the window (rows written by pool_key_blocks)."""
-    _cuda(q, k_pool, v_pool, req_to_token, req_pool_indices, sinks, slopes)
+    and value per block of `size` tokens that lies wholly before the window (rows written by pool_key_blocks).
+    keep_first: positions below it stay visible when the window has moved past them.  dist_bias fp32 [heads, len]:
+    dist_bias[h, min(distance, len − 1)] joins the score."""
+    _cuda(q, k_pool, v_pool, req_to_token, req_pool_indices, sinks, slopes, dist_bias)
+    if dist_bias is not None and (dist_bias.dtype != torch.float32 or not dist_bias.is_contiguous() or dist_bias.dim() != 2
+                                  or dist_bias.shape[0] != num_q_heads):
+        raise RuntimeError("attn_general: dist_bias is contiguous fp32 [heads, distances]")
     T = q.shape[0]
     if q.dim() != 2 or q.stride(1) != 1:
         raise RuntimeError("attn_general: q must be [T, H * head_dim] with contiguous rows")
@@ -934,13 +959,14 @@ def attn_general(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, re
             raise RuntimeError("attn_general: sinks and slopes are fp32")
     out = torch.empty((T, num_q_heads * v_dim), device=q.device, dtype=q.dtype)
     size, run_len, base = blocks or (0, 0, 0)
-    check(lib.spd_attn_general_blocks(out.data_ptr(), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
+    check(lib.spd_attn_general_keys(out.data_ptr(), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
                                   req_to_token.data_ptr(), req_pool_indices.data_ptr(), _ptr(seq_lens), _ptr(prefix_lens),
                                   _ptr(extend_lens), _ptr(extend_start_loc), req_pool_indices.numel(), T, num_q_heads,
                                   num_kv_heads, head_dim, v_dim, q.stride(0), out.stride(0), req_to_token.stride(0),
                                   float(sm_scale), int(window), _ptr(sinks), _ptr(slopes), float(qtemp_coef),
                                   int(qtemp_every), int(max_extend_len), float(softcap or 0.0), int(num_v_heads),
-                                  int(v_slot_stride), int(size), int(run_len), int(base), _dta(q), _stream()),
+                                  int(v_slot_stride), int(size), int(run_len), int(base), int(keep_first), _ptr(dist_bias),
+                                  dist_bias.shape[1] if dist_bias is not None else 0, _dta(q), _stream()),
           "spd_attn_general")
     return out
 
@@ -1158,21 +1184,24 @@ def residual_tanh_norm(x: torch.Tensor, weight: Optional[torch.Tensor], bias: Op
 def rotary_segment(src: torch.Tensor, dst: torch.Tensor, heads: int, head_dim: int, rot: int = 0,
                    bias: Optional[torch.Tensor] = None, src_head: Optional[int] = None, dst_head: Optional[int] = None,
                    to_pool: bool = False, norm_eps: Optional[float] = None,
-                   norm_weight: Optional[torch.Tensor] = None) -> _lib.RotarySegment:
+                   norm_weight: Optional[torch.Tensor] = None, norm_row: bool = False) -> _lib.RotarySegment:
     """One piece of rotary_segments: src / dst are 2-D views whose first element is the first head's first channel
     (row stride = stride(0); src_head / dst_head default to head_dim).  norm_eps (not None): every head is brought to
-    unit RMS over its channels after the bias and before the rotation, times norm_weight (fp32 [head_dim], optional)."""
+    unit RMS over its channels after the bias and before the rotation, times norm_weight (fp32 [head_dim], optional).
+    norm_row: the norm runs over all heads together instead, norm_weight [heads · head_dim]."""
     _cuda(src, dst, bias, norm_weight)
     if norm_weight is not None and (norm_eps is None or norm_weight.dtype != torch.float32
-                                    or not norm_weight.is_contiguous() or norm_weight.numel() != head_dim):
-        raise RuntimeError("rotary_segment: norm_weight is contiguous fp32 [head_dim], with norm_eps")
+                                    or not norm_weight.is_contiguous()
+                                    or norm_weight.numel() != (heads * head_dim if norm_row else head_dim)):
+        raise RuntimeError("rotary_segment: norm_weight is contiguous fp32 [head_dim] (norm_row: [heads * head_dim]), with "
+                           "norm_eps")
     if src.stride(-1) != 1 or dst.stride(-1) != 1 or src.dtype != dst.dtype:
         raise RuntimeError("rotary_segment: src and dst have contiguous rows and one dtype")
     if bias is not None and (bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() != heads * head_dim):
         raise RuntimeError("rotary_segment: bias is contiguous fp32 [heads * head_dim]")
     seg = _lib.RotarySegment(src.data_ptr(), _ptr(bias), dst.data_ptr(), src.stride(0), dst.stride(0), heads, head_dim, rot,
                              head_dim if src_head is None else src_head, head_dim if dst_head is None else dst_head,
-                             1 if to_pool else 0, _ptr(norm_weight), 0 if norm_eps is None else 1,
+                             1 if to_pool else 0, _ptr(norm_weight), 0 if norm_eps is None else (2 if norm_row else 1),
                              0.0 if norm_eps is None else float(norm_eps))
     seg.keep = (src, dst, bias, norm_weight)  # the descriptor holds raw pointers: the tensors live as long as it does
     return seg

@@ -15,6 +15,7 @@ _MODELS: Dict[str, Tuple[str, str]] = {
     "matepel": ("matepel", "MatepelForCausalLM"),
     "sugelix": ("sugelix", "SugelixForCausalLM"),
     "fudonex": ("fudonex", "FudonexForCausalLM"),
+    "kuforax": ("kuforax", "KuforaxForCausalLM"),
 }
 
 
