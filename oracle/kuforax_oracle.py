@@ -99,8 +99,8 @@ def distance_bucket(n, rows, far):
     """Row of the bias table for a key n tokens back: one row per distance below rows // 2, then rows that are spaced by
     the logarithm of the distance, reaching the last one at `far`."""
     half = rows // 2
-    if n < half:
-        return n
+    if n < half or rows == 1:
+        return min(n, rows - 1)
     at = math.log(n / half) / math.log(far / half) * (rows - half)
     return min(rows - 1, half + math.floor(at + 1e-9))  # (1e-9: a power that is an integer on paper)
 
@@ -178,17 +178,24 @@ def route(z, correction, top, groups=None):
 
 
 def routing_margin(z, correction, top, groups=None):
-    """How far the choice is from another one, per token (in score units): between the last chosen and the first not
-    chosen expert, and between the last kept and the first dropped group."""
+    """How far the choice is from another one, per token: the least (c_i - c_j) / (s_i + s_j) over pairs of a chosen and a
+    not chosen expert, and of the best experts of a kept and a dropped group — the relative change of scores that swaps
+    them."""
     s, c = choice_scores(z, correction, groups)
-    inf = torch.full(c.shape[:1], float("inf"), dtype=F64)
-    margin = inf
-    if top < c.shape[-1]:
-        val = torch.topk(c, top + 1, dim=-1).values
-        margin = val[:, top - 1] - val[:, top]
+    idx, _ = route(z, correction, top, groups)
+    chosen = torch.zeros_like(c, dtype=torch.bool).scatter_(1, idx, True)
+    open_ = torch.isfinite(c)
+
+    def least(value, score, a, b):
+        pair = (value[:, :, None] - value[:, None, :]) / (score[:, :, None] + score[:, None, :])
+        return pair.masked_fill(~(a[:, :, None] & b[:, None, :]), float("inf")).flatten(1).min(1).values
+
+    margin = least(c.masked_fill(~open_, 0.0), s, chosen, open_ & ~chosen)
     if groups and int(groups["keep"]) < int(groups["count"]):
-        g = torch.topk((s + f64(correction)).view(len(c), int(groups["count"]), -1).max(-1).values, int(groups["keep"]) + 1)
-        margin = torch.minimum(margin, g.values[:, -2] - g.values[:, -1])
+        n = int(groups["count"])
+        best, at = (s + f64(correction)).view(len(c), n, -1).max(-1)
+        kept = open_.view(len(c), n, -1).any(-1)
+        margin = torch.minimum(margin, least(best, s.view(len(c), n, -1).gather(-1, at[..., None])[..., 0], kept, ~kept))
     return margin
 
 
@@ -243,6 +250,18 @@ def forward(cfg, W, tokens, want_layers=False, margins: Optional[list] = None):
         layers.append(x.clone())
     logits = linear(rms_norm_around_one(x, W["final.norm"], eps), W["head"])
     return (logits, torch.stack(layers)) if want_layers else logits
+
+
+class Stepper:
+    """Token-by-token use of the whole-sequence statement: keeps the tokens fed so far and recomputes."""
+
+    def __init__(self, cfg, W):
+        self.cfg, self.W, self.tokens = cfg, W, []
+
+    def feed(self, tokens):
+        """→ logits of the tokens just fed [len(tokens), vocab]."""
+        self.tokens += list(tokens)
+        return forward(self.cfg, self.W, self.tokens)[-len(tokens):]
 
 
 # ---- configurations and random checkpoints for the tests ----------------------------------------------------

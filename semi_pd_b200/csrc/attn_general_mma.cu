@@ -130,6 +130,10 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
     nbx[x] = !ok ? 0 : kb.size > 0 ? (int)key_blocks_seen(kb, pi[x], window) : (kb.keep <= hi[x] ? kb.keep : hi[x] + 1);
     lo[x] = window > 0 && pi[x] - window + 1 > j_lo ? NB + (int)(pi[x] - window + 1 - j_lo) : NB;
   }
+  // entries that all 16 rows of this warp see (none where a row lies past the portion)
+  const int64_t w_first = i0 + warp * 16, w_last = w_first + 15;
+  const int full_hi = w_last <= j_hi ? NB + (int)(w_first - j_lo) : -1;
+  const int full_lo = window > 0 && w_last - window + 1 > j_lo ? NB + (int)(w_last - window + 1 - j_lo) : NB;
   float sc[2], scc[2];  // score multipliers into the exp2 domain, and (with a cap) into units of the cap
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
@@ -186,6 +190,17 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
     }
     const int eb = t * kGmBK;
     float mx[2] = {-INFINITY, -INFINITY};
+    if (softcap > 0.f) {
+#pragma unroll
+      for (int nb = 0; nb < kGmBK / 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nb][e] = capl * gm_tanh(s[nb][e] * scc[e >> 1]);
+    } else {
+#pragma unroll
+      for (int nb = 0; nb < kGmBK / 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nb][e] *= sc[e >> 1];
+    }
     if (brow != nullptr) {
       // rows x = 0, 1 are eight apart, columns of neighbouring nb too: row 1 of nb has the distance of row 0 of nb - 1
       float bt[kGmBK / 8 + 1][2];
@@ -203,18 +218,29 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int x = e >> 1;
-          const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
+          const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);  // (its mask follows)
           float b = bt[nb + 1 - x][e & 1];
           if (eb < NB && idx < NB && gap > 0) {
             const int64_t d = pi[x] - idx;
             b = brow[d < db.len ? d : db.len - 1];
           }
-          const bool ok = (idx >= lo[x] && idx <= hi[x]) || idx < nbx[x];
-          const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc[x]) : s[nb][e] * sc[x];
-          const float v = ok ? fmaf(b, kLog2e, z) - sl * (float)(hi[x] - idx + (idx < NB ? gap : 0)) : -INFINITY;
-          s[nb][e] = v;
-          mx[x] = fmaxf(mx[x], v);
+          s[nb][e] = fmaf(b, kLog2e, s[nb][e]);
         }
+    }
+    if (sl != 0.f) {
+#pragma unroll
+      for (int nb = 0; nb < kGmBK / 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
+          s[nb][e] -= sl * (float)(hi[e >> 1] - idx + (idx < NB ? gap : 0));
+        }
+    }
+    if (eb >= full_lo && eb + kGmBK - 1 <= full_hi) {  // every row of the warp sees the whole tile
+#pragma unroll
+      for (int nb = 0; nb < kGmBK / 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[nb][e]);
     } else {
 #pragma unroll
       for (int nb = 0; nb < kGmBK / 8; ++nb)
@@ -223,10 +249,8 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
           const int x = e >> 1;
           const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
           const bool ok = (idx >= lo[x] && idx <= hi[x]) || idx < nbx[x];
-          const float z = softcap > 0.f ? capl * gm_tanh(s[nb][e] * scc[x]) : s[nb][e] * sc[x];
-          const float v = ok ? z - sl * (float)(hi[x] - idx + (idx < NB ? gap : 0)) : -INFINITY;
-          s[nb][e] = v;
-          mx[x] = fmaxf(mx[x], v);
+          s[nb][e] = ok ? s[nb][e] : -INFINITY;
+          mx[x] = fmaxf(mx[x], s[nb][e]);
         }
     }
     float ms[2];

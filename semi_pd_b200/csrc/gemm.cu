@@ -445,7 +445,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUt
           tmem_ld_wait();
 #pragma unroll
           for (int j = 0; j < kChunk; ++j)
-            v[j] = kEpi == SPD_EPI_GELU ? gelu_f32(to_f32<T>(from_f32<T>(__uint_as_float(r[j])))) : __uint_as_float(r[j]);
+            v[j] = kEpi == SPD_EPI_GELU ? gelu_fast_f32(to_f32<T>(from_f32<T>(__uint_as_float(r[j])))) : __uint_as_float(r[j]);
         }
         store_chunk(xt, yt, c, v);
       }
@@ -815,7 +815,10 @@ int spd_gemm_grouped(void* C, const void* A, const void* W, int64_t M, int64_t N
       if ((rc = get_tmap(&ty, W, static_cast<uint64_t>(num_groups) * 2 * N, K, ldw, BN / 2))) return rc;
       SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, BN, false, SPD_EPI_SILU_MUL>(tx, ty, p, grid, st); });
     }
-    constexpr int BN = 128;
+    // 128 x 256 tiles where they pad N no more than 128 x 128 ones by an eighth and still fill the SMs
+    const int64_t pad256 = (N + 255) / 256 * 256, pad128 = (N + 127) / 128 * 128;
+    const bool use256 = w_group_col_stride == 0 && pad256 - pad128 <= N / 8 && p.x_tiles * (pad256 / 256) >= sms;
+    const int BN = use256 ? 256 : 128;
     p.y_tiles = static_cast<int>((N + BN - 1) / BN);
     const int total = p.x_tiles * p.y_tiles;
     const int grid = total < sms ? total : sms;
@@ -830,9 +833,12 @@ int spd_gemm_grouped(void* C, const void* A, const void* W, int64_t M, int64_t N
       p.y_group_rows = N;
       if ((rc = get_tmap(&ty, W, static_cast<uint64_t>(num_groups) * N, K, ldw, BN))) return rc;
     }
-    if (epilogue == SPD_EPI_GELU)
-      SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, BN, false, SPD_EPI_GELU>(tx, ty, p, grid, st); });
-    SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, BN, false, SPD_EPI_NONE>(tx, ty, p, grid, st); });
+    if (epilogue == SPD_EPI_GELU) {
+      if (use256) SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, 256, false, SPD_EPI_GELU>(tx, ty, p, grid, st); });
+      SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, 128, false, SPD_EPI_GELU>(tx, ty, p, grid, st); });
+    }
+    if (use256) SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, 256, false, SPD_EPI_NONE>(tx, ty, p, grid, st); });
+    SPD_DISPATCH_DTYPE(dtype, { return launch_gemm<T, 128, false, SPD_EPI_NONE>(tx, ty, p, grid, st); });
   }
   // cols mode (block diagonal): C[:, g*N:(g+1)*N] = A[:, g*a_group_stride : +K] * W[g*N:(g+1)*N, :K]^T
   SPD_REQUIRE(epilogue == SPD_EPI_NONE && w_group_col_stride == 0, SPD_E_BADARG,

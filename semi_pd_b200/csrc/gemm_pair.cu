@@ -236,7 +236,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           tmem_ld_wait();
 #pragma unroll
           for (int j = 0; j < 32; ++j)
-            v[j] = kEpi == SPD_EPI_GELU ? gelu_f32(to_f32<T>(from_f32<T>(__uint_as_float(r[j])))) : __uint_as_float(r[j]);
+            v[j] = kEpi == SPD_EPI_GELU ? gelu_fast_f32(to_f32<T>(from_f32<T>(__uint_as_float(r[j])))) : __uint_as_float(r[j]);
         }
         const int64_t n0 = static_cast<int64_t>(yt) * kBNOut + c;
         if (m < p.m_rows) {

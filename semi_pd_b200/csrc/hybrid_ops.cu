@@ -223,7 +223,8 @@ constexpr int kRouteMaxGroups = 32;
 // scores s = sigmoid(z) or softmax(z); selection runs on the biased score c = s + correction.  With groups the
 // experts are cut into equal runs of neighbours, every run is ranked by its largest biased score or (group_top 2)
 // its two largest added together, and experts outside the keep_groups highest-ranked runs are ineligible (c = -inf there).  The weight of a
-// selected expert is its unbiased s (optionally renormalised).
+// selected expert is its unbiased s (optionally renormalised).  A lane holds PER experts.
+template <int PER>
 __global__ void __launch_bounds__(128)
 moe_route_scores_kernel(int32_t* __restrict__ topk_ids, float* __restrict__ topk_w, const float* __restrict__ logits,
                         int64_t ld, int64_t tokens, int E, int k, int score_func, int renorm, float scale,
@@ -233,7 +234,6 @@ moe_route_scores_kernel(int32_t* __restrict__ topk_ids, float* __restrict__ topk
   const int lane = threadIdx.x & 31;
   const int64_t t = blockIdx.x * 4ll + (threadIdx.x >> 5);
   if (t >= tokens) return;
-  constexpr int PER = kRouteMaxExperts / 32;
   float v[PER];  // scores (0 outside the experts)
   if (score_func == 1) {
 #pragma unroll
@@ -581,7 +581,11 @@ int spd_moe_route_scores(int32_t* topk_ids, float* topk_w, const float* logits, 
               SPD_E_SHAPE, "spd_moe_route_scores: %d groups (max %d, dividing the experts), keep %d", num_groups,
               kRouteMaxGroups, keep_groups);
   if (tokens == 0) return 0;
-  SPD_CUDA(launch(moe_route_scores_kernel, dim3((unsigned)((tokens + 3) / 4)), dim3(128), 0, as_stream(stream),
+  auto kern = num_experts <= 32    ? moe_route_scores_kernel<1>
+              : num_experts <= 64  ? moe_route_scores_kernel<2>
+              : num_experts <= 128 ? moe_route_scores_kernel<4>
+                                   : moe_route_scores_kernel<kRouteMaxExperts / 32>;
+  SPD_CUDA(launch(kern, dim3((unsigned)((tokens + 3) / 4)), dim3(128), 0, as_stream(stream),
                   pdl_enabled(), topk_ids, topk_w, logits, ld, tokens, num_experts, top_k, score_func, renormalize,
                   scale, correction, num_groups, keep_groups, group_top));
   return 0;

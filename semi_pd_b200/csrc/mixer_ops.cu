@@ -495,6 +495,142 @@ rotary_segments_rownorm_kernel(RotarySegments segs, const int64_t* __restrict__ 
   }
 }
 
+// The same in 16-byte pieces that stay in registers between the sum and the rotation (half-split layout; head_dim, rot / 2,
+// strides multiples of the vector width; weights, biases and table rows 16-byte aligned).  The items of all segments form
+// one list — per head rot / (2 N) vectors that carry their rotation partner, then (head_dim - rot) / N single ones — of
+// which a thread owns NI.
+struct RowNormItems {
+  int start[5];  // first item of each segment; start[n] = all items
+};
+template <typename T, int NI>
+__global__ void __launch_bounds__(kRowNormThreads)
+rotary_segments_rownorm_vec_kernel(RotarySegments segs, RowNormItems items, const int64_t* __restrict__ positions,
+                                   const int64_t* __restrict__ loc, const float* __restrict__ cos_sin, int rot_max,
+                                   int64_t max_positions) {
+  griddep_wait();
+  griddep_launch_dependents();
+  constexpr int N = Vec16<T>::kN;
+  __shared__ float red[4][kRowNormThreads / 32];
+  const int64_t t = blockIdx.x;
+  int seg_of[NI], col[NI];  // segment (-1: none), first channel within the row of heads
+  Vec16<T> va[NI], vb[NI];
+  float ss[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int u = 0; u < NI; ++u) {
+    int item = (int)(threadIdx.x + u * blockDim.x);
+    int s = 0;
+    while (s < segs.n && item >= items.start[s + 1]) ++s;
+    seg_of[u] = s < segs.n ? s : -1;
+    if (s >= segs.n) continue;
+    const RotarySegment& sg = segs.seg[s];
+    item -= items.start[s];
+    const int leads = sg.rot / (2 * N), per_head = leads + (sg.head_dim - sg.rot) / N;
+    const int h = item / per_head, x = item - h * per_head;
+    const int d0 = x < leads ? x * N : sg.rot + (x - leads) * N;
+    col[u] = h * sg.head_dim + d0;
+    const T* sp = reinterpret_cast<const T*>(sg.src) + t * sg.src_row + h * sg.src_head + d0;
+    va[u] = ldv(sp);
+    if (x < leads) vb[u] = ldv(sp + (sg.rot >> 1));
+    if (x >= leads) seg_of[u] |= 8;  // no partner
+  }
+  int64_t p = positions[t];
+  p = p < 0 ? 0 : (p < max_positions ? p : max_positions - 1);
+  const float* cs = cos_sin != nullptr ? cos_sin + p * rot_max : nullptr;
+  const int half_max = rot_max >> 1;
+  const int64_t slot = loc != nullptr ? loc[t] : 0;
+  auto with_vector = [&](const Vec16<T>& v, const float* bias, int c, float (&x)[N]) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) x[i] = to_f32<T>(v.e()[i]);
+    if (bias != nullptr) {
+#pragma unroll
+      for (int i = 0; i < N; i += 4) {
+        const float4 b = *reinterpret_cast<const float4*>(bias + c + i);
+        x[i] += b.x; x[i + 1] += b.y; x[i + 2] += b.z; x[i + 3] += b.w;
+      }
+    }
+  };
+#pragma unroll
+  for (int u = 0; u < NI; ++u) {
+    if (seg_of[u] < 0) continue;
+    const RotarySegment& sg = segs.seg[seg_of[u] & 3];
+    if (sg.norm != 2) continue;
+    float x[N], sum = 0.f;
+    with_vector(va[u], sg.bias, col[u], x);
+#pragma unroll
+    for (int i = 0; i < N; ++i) sum = fmaf(x[i], x[i], sum);
+    if ((seg_of[u] & 8) == 0) {
+      with_vector(vb[u], sg.bias, col[u] + (sg.rot >> 1), x);
+#pragma unroll
+      for (int i = 0; i < N; ++i) sum = fmaf(x[i], x[i], sum);
+    }
+#pragma unroll
+    for (int s = 0; s < 4; ++s) ss[s] += (seg_of[u] & 3) == s ? sum : 0.f;
+  }
+#pragma unroll
+  for (int s = 0; s < 4; ++s) {
+    if (s >= segs.n || segs.seg[s].norm != 2) continue;
+    ss[s] = warp_sum(ss[s]);
+    if ((threadIdx.x & 31) == 0) red[s][threadIdx.x >> 5] = ss[s];
+  }
+  __syncthreads();
+  const int warps = blockDim.x >> 5;
+#pragma unroll
+  for (int u = 0; u < NI; ++u) {
+    if (seg_of[u] < 0) continue;
+    const int s = seg_of[u] & 3;
+    const RotarySegment& sg = segs.seg[s];
+    float inv = 1.f;
+    const float* nw = nullptr;
+    if (sg.norm == 2) {
+      float sum = 0.f;
+      for (int i = 0; i < warps; ++i) sum += red[s][i];
+      inv = 1.0f / sqrtf(sum / (float)(sg.heads * sg.head_dim) + sg.norm_eps);
+      nw = sg.norm_w;
+    }
+    const int half = sg.rot >> 1;
+    const int h = col[u] / sg.head_dim, d0 = col[u] - h * sg.head_dim;
+    T* dp = reinterpret_cast<T*>(sg.dst) + (sg.to_pool ? slot : t) * sg.dst_row + h * sg.dst_head + d0;
+    auto scaled = [&](const Vec16<T>& v, int c, float (&x)[N]) {
+      with_vector(v, sg.bias, c, x);
+#pragma unroll
+      for (int i = 0; i < N; ++i) x[i] *= inv;
+      if (nw != nullptr) {
+#pragma unroll
+        for (int i = 0; i < N; i += 4) {
+          const float4 w = *reinterpret_cast<const float4*>(nw + c + i);
+          x[i] *= w.x; x[i + 1] *= w.y; x[i + 2] *= w.z; x[i + 3] *= w.w;
+        }
+      }
+    };
+    float a[N];
+    Vec16<T> o;
+    scaled(va[u], col[u], a);
+    if ((seg_of[u] & 8) == 0) {
+      float b[N];
+      Vec16<T> ob;
+      scaled(vb[u], col[u] + half, b);
+#pragma unroll
+      for (int i = 0; i < N; i += 4) {
+        const float4 c4 = *reinterpret_cast<const float4*>(cs + d0 + i);
+        const float4 s4 = *reinterpret_cast<const float4*>(cs + half_max + d0 + i);
+        const float c[4] = {c4.x, c4.y, c4.z, c4.w}, sn[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float x = a[i + e], y = b[i + e];
+          a[i + e] = x * c[e] - y * sn[e];
+          b[i + e] = y * c[e] + x * sn[e];
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < N; ++i) ob.e()[i] = from_f32<T>(b[i]);
+      stv(dp + half, ob);
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) o.e()[i] = from_f32<T>(a[i]);
+    stv(dp, o);
+  }
+}
+
 // The residual update of a layer that norms its sublayer's output: x[row] += y / rms(y) * coef (y null: no update),
 // then out = x in T, or (w given) x / rms(x) * (off + w).  One CTA per row; a row of up to NV vectors per thread stays
 // in registers (VEC = 1: any size, read twice).
@@ -756,6 +892,26 @@ int spd_rotary_segments(const spd_rotary_segment_t* segments, int num_segments, 
   }
   if (row_norm) {
     SPD_REQUIRE(!head_norm, SPD_E_BADARG, "spd_rotary_segments: norms per head and per row in one launch");
+    bool pieces = vec && !paired && rot_max % 8 == 0 && aligned16(cos_sin);
+    RowNormItems items{};
+    for (int i = 0; i < num_segments; ++i) {
+      const RotarySegment& s = segs.seg[i];
+      pieces = pieces && aligned16(s.bias) && aligned16(s.norm_w);
+      items.start[i + 1] = items.start[i] + s.heads * (s.rot / (2 * vecn) + (s.head_dim - s.rot) / vecn);
+    }
+    const int total = items.start[num_segments];
+    if (pieces && total <= 4 * kRowNormThreads) {
+      const int ni = total <= kRowNormThreads ? 1 : total <= 2 * kRowNormThreads ? 2 : 4;
+      const int threads = ((total + ni - 1) / ni + 31) / 32 * 32;
+      SPD_DISPATCH_ANY(dtype, {
+        auto kern = ni == 1   ? rotary_segments_rownorm_vec_kernel<T, 1>
+                    : ni == 2 ? rotary_segments_rownorm_vec_kernel<T, 2>
+                              : rotary_segments_rownorm_vec_kernel<T, 4>;
+        SPD_CUDA(launch(kern, dim3((unsigned)tokens), dim3((unsigned)threads), 0, as_stream(stream), pdl_enabled(), segs,
+                        items, positions, loc, cos_sin, rot_max, max_positions));
+      });
+      return 0;
+    }
     SPD_DISPATCH_ANY(dtype, {
       auto kern = vec ? rotary_segments_rownorm_kernel<T, 16 / (int)sizeof(T)> : rotary_segments_rownorm_kernel<T, 1>;
       SPD_CUDA(launch(kern, dim3((unsigned)tokens), dim3(kRowNormThreads), 0, as_stream(stream), pdl_enabled(), segs,
