@@ -261,7 +261,7 @@ int64_t spd_comm_max_bytes(const spd_comm_t* comm);
 int spd_comm_status(spd_comm_t* comm, int* timed_out);
 int spd_allreduce(spd_comm_t* comm, void* out, const void* in, int64_t count, int dtype, int algo,
                   spd_stream_t stream);
-/* The all-reduce fused with its consumer (round 2): x = sum over ranks of in[rows, dim];
+/* The all-reduce fused with its consumer: x = sum over ranks of in[rows, dim];
  * residual += x (rounded to the dtype as fused_add_rmsnorm stores it); out = RMSNorm(residual) * weight
  * — S/layers/linear.py:1265-1266 (tensor_model_parallel_all_reduce after o_proj / down_proj)
  * followed by S/layers/layernorm.py:46-57 (fused_add_rmsnorm) in ONE kernel over the peer-mapped

@@ -1,5 +1,5 @@
 """CPU oracle for BASELINE configs[3] (DeepSeek-V2-Lite: MLA attention + MoE) — TEST INFRASTRUCTURE
-ONLY, prepared for the next round: no CUDA path exists for this model yet.
+ONLY.
 
 Restates, in fp32 torch, what the reference computes (infinigence/Semi-PD @ 2565f9f, paths relative
 to python/sglang/srt/):

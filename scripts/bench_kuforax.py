@@ -153,18 +153,26 @@ def kernel_table(z, flush):
             xs = ops.moe_gather_scaled(a, row_token, inv_pos, None)
             tiles = float((tile_group >= 0).sum()) * 128
             if not like:
-                ms = ev(lambda: ops.linear_grouped_any(xs, up, tile_group, E, F, gelu=True))
-                add(f"grouped GEMM + GELU {n}x{k} rows ({tiles:.0f} in tiles) {F}x{Wd}", "", ms, flops=2.0 * rows_used * F * Wd,
-                    bytes_=None) if n == T else add(f"grouped GEMM + GELU B={n} {F}x{Wd}", "", ms, bytes_=E * F * Wd * 2)
+                for act, note in ((True, ""), (False, "like: GELU in the epilogue")):
+                    ms = ev(lambda: ops.linear_grouped_any(xs, up, tile_group, E, F, gelu=act))
+                    name = "grouped GEMM" + (" + GELU" if act else "")
+                    if n == T:
+                        add(f"{name} {n}x{k} rows ({tiles:.0f} in tiles) {F}x{Wd}", note, ms, flops=2.0 * rows_used * F * Wd)
+                    else:
+                        add(f"{name} B={n} {F}x{Wd}", note, ms, bytes_=E * F * Wd * 2)
             else:
                 gu = torch.cat([up, up], 0)
                 ms = ev(lambda: ops.linear_grouped_any(xs, gu, tile_group, E, F, silu_mul=True))
-                add(f"grouped GEMM + SiLU mul {n}x{k} rows {F}x{Wd}", "like: GELU in the epilogue", ms,
-                    flops=4.0 * rows_used * F * Wd) if n == T else add(
-                        f"grouped GEMM + SiLU mul B={n} {F}x{Wd}", "like: GELU in the epilogue", ms, bytes_=2 * E * F * Wd * 2)
+                if n == T:
+                    add(f"grouped GEMM + SiLU mul {n}x{k} rows {F}x{Wd}", "like: GELU in the epilogue", ms,
+                        flops=4.0 * rows_used * F * Wd)
+                else:
+                    add(f"grouped GEMM + SiLU mul B={n} {F}x{Wd}", "like: GELU in the epilogue", ms, bytes_=2 * E * F * Wd * 2)
     a, su = r_(T, Wd), r_(2 * F, Wd)
     ms = ev(lambda: ops.linear_gelu_any(a, su[:F]))
     add(f"GEMM + GELU {T}x{F}x{Wd}", "", ms, flops=2.0 * T * F * Wd)
+    ms = ev(lambda: ops.linear_any(a, su[:F]))
+    add(f"GEMM {T}x{F}x{Wd}", "like: GELU in the epilogue", ms, flops=2.0 * T * F * Wd)
     ms = ev(lambda: ops.linear_silu_mul_any(a, su))
     add(f"GEMM + SiLU mul {T}x{F}x{Wd}", "like: GELU in the epilogue", ms, flops=4.0 * T * F * Wd)
     return rows

@@ -35,7 +35,7 @@
 // consecutive (and the tile is full); anything else — a foreign req_to_token, the reference
 // allocator's scattered slots, the ragged last tile of a sequence — takes the gather path:
 // 16-byte cp.async per row chunk through req_to_token into the same swizzled layout.
-// (tile::gather4, 4 rows x 128 B per instruction, was built and measured in round 1: correct,
+// (tile::gather4, 4 rows x 128 B per instruction, was built and measured: correct,
 // but ~1 instruction per 27 clk per SM -> 36 GB/s per SM, below the cp.async gather's 47;
 // profiles/r01_decode_attention_loader_experiments.md.)
 #include <cuda.h>

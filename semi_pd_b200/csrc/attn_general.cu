@@ -468,15 +468,25 @@ int attn_general_decode_group_launch(size_t smem, int q_bytes, int64_t batch, cu
   return 0;
 }
 
-template <typename T>
+// VEC elements at a time: every row a multiple of VEC, aligned to VEC elements
+template <typename T, int VEC>
+struct alignas(sizeof(T) * VEC) StoreVec {
+  T e[VEC];
+};
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 kv_store_kernel(const T* __restrict__ k, const T* __restrict__ v, T* __restrict__ k_pool, T* __restrict__ v_pool,
                 const int64_t* __restrict__ loc, int64_t k_row, int64_t v_row, int64_t k_stride, int64_t v_stride) {
   const int64_t t = blockIdx.x;
   const int64_t slot = loc[t];
-  for (int64_t i = threadIdx.x; i < k_row; i += 256) k_pool[slot * k_row + i] = k[t * k_stride + i];
-  if (v != nullptr)
-    for (int64_t i = threadIdx.x; i < v_row; i += 256) v_pool[slot * v_row + i] = v[t * v_stride + i];
+  using V = StoreVec<T, VEC>;
+  const int64_t n = v != nullptr ? k_row + v_row : k_row;
+  for (int64_t i = threadIdx.x * (int64_t)VEC; i < n; i += blockDim.x * (int64_t)VEC) {
+    if (i < k_row)
+      *reinterpret_cast<V*>(k_pool + slot * k_row + i) = *reinterpret_cast<const V*>(k + t * k_stride + i);
+    else
+      *reinterpret_cast<V*>(v_pool + slot * v_row + (i - k_row)) = *reinterpret_cast<const V*>(v + t * v_stride + (i - k_row));
+  }
 }
 
 // Block rows of the blocks that a batch completes: the mean over the block's cache rows of K and V, as the cache holds
@@ -586,7 +596,13 @@ int spd_kv_store(const void* k, const void* v, void* k_pool, void* v_pool, const
   SPD_REQUIRE(tokens >= 0 && k_row_elems > 0 && v_row_elems >= 0, SPD_E_BADARG, "spd_kv_store: bad sizes");
   if (tokens == 0) return 0;
   SPD_DISPATCH_ANY(dtype, {
-    SPD_CUDA(launch(kv_store_kernel<T>, dim3((unsigned)tokens), dim3(256), 0, as_stream(stream), /*pdl=*/false,
+    constexpr int N = 16 / (int)sizeof(T);
+    const bool vec = k_row_elems % N == 0 && k_stride % N == 0 && aligned16(k) && aligned16(k_pool) &&
+                     (v == nullptr || (v_row_elems % N == 0 && v_stride % N == 0 && aligned16(v) && aligned16(v_pool)));
+    const int64_t items = (k_row_elems + (v != nullptr ? v_row_elems : 0)) / (vec ? N : 1);
+    const unsigned threads = (unsigned)(items < 256 ? (items + 31) / 32 * 32 : 256);
+    auto kern = vec ? kv_store_kernel<T, N> : kv_store_kernel<T, 1>;
+    SPD_CUDA(launch(kern, dim3((unsigned)tokens), dim3(threads), 0, as_stream(stream), /*pdl=*/false,
                     (const T*)k, (const T*)v, (T*)k_pool, (T*)v_pool, loc, k_row_elems, v_row_elems, k_stride,
                     v_stride));
   });

@@ -13,7 +13,7 @@
 // One CTA = one query token x one group of 16 heads x one KV split.  Both products run on the
 // tensor cores through warp-level mma.sync m16n8k16 (M = the 16 heads): this is the first MLA
 // kernel of the repo; the tcgen05 swap-AB form of attn_decode.cu with N = 16 real heads is the
-// planned successor (DESIGN.md).  Per 32-token chunk:
+// planned successor.  Per 32-token chunk:
 //   K rows (= V rows) -> smem by 16-byte cp.async through req_to_token, double buffered;
 //   S[16 x 32]  = Q[16 x DL] K^T      k-steps split over the 8 warps, partials reduced in smem;
 //   online softmax, one warp per pair of heads, exp2 domain;

@@ -398,7 +398,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         mbar_wait(q_full, itn & 1);
         // S_w(j, h): the warpgroup's previous P in these columns has been consumed by PV(j-1, h),
         // issued earlier by this thread — tcgen05.mma executes in issue order.
-        // (Tried in round 2: interleaving the two warpgroups' MMAs instruction by instruction —
+        // (Tried: interleaving the two warpgroups' MMAs instruction by instruction —
         // back-to-back tcgen05.mma on ONE accumulator cost ~43 clk (SS) / ~10 clk (TS) more than
         // N/2 each, alternating accumulators runs at the shared-memory operand rate,
         // profiles/r02_tcgen05_2cta_probe.log.  The issuer's time per unit pair did drop from
@@ -578,7 +578,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     uint32_t tn = 0;
     const bool tracer = kTrace && (threadIdx.x & 127) == 0;
     // ---- epilogue: O / l, TMEM -> registers -> global ----
-    // (Tried in round 2: DEFERRING it until the next item's first unit has been exponentiated, so
+    // (Tried: DEFERRING it until the next item's first unit has been exponentiated, so
     // that the ~1500-1900 clk drain of the item's last PV is spent on useful work.  The drain wait
     // did shrink to ~700 clk, but o_free — and with it the next item's first PV — moved later by
     // a whole softmax pass, and the kernel got 5 % slower at 8 x 1024; not kept.)
@@ -594,7 +594,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const float inv_l = e_l > 0.f ? 1.f / e_l : 0.f;
       // A full tile leaves through shared memory and one TMA store per 64-column block: with one
       // thread per row, direct 16-byte stores touch 32 different lines per warp instruction and
-      // the 128 rows x 256 B took ~5900 clk per item (in-kernel timeline, round 2) — a quarter of
+      // the 128 rows x 256 B took ~5900 clk per item (in-kernel timeline) — a quarter of
       // the kernel at 1024-token prompts.  A ragged last tile (fewer than 128 rows) must not write
       // the rows of the next request and keeps the direct path.
       const bool full_tile = e_rows == kPfM;

@@ -203,7 +203,7 @@ class ModelRunner:
             return
         if self.tp_size > 1 and (self.tp_comm is None or self.tp_comm.max_bytes == 0):
             # only libspd's peer-memory collectives are captured (torch.distributed's NCCL
-            # all-reduce inside the decode graph hung on the pool in round 1)
+            # all-reduce inside the decode graph has hung)
             logger.warning("TP > 1 without the libspd communicator: decode CUDA graphs disabled")
             return
         self.cuda_graph_runner = CudaGraphRunner(self)
