@@ -213,19 +213,22 @@ attn_general_mma_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
           d = d < 0 ? 0 : (d < db.len ? d : db.len - 1);  // (a negative distance is masked below)
           bt[i][p] = brow[d];
         }
+      if (eb < NB && gap > 0) {  // kept tokens in front of the window: element by element
 #pragma unroll
-      for (int nb = 0; nb < kGmBK / 8; ++nb)
+        for (int nb = 0; nb < kGmBK / 8; ++nb)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int x = e >> 1;
-          const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);  // (its mask follows)
-          float b = bt[nb + 1 - x][e & 1];
-          if (eb < NB && idx < NB && gap > 0) {
-            const int64_t d = pi[x] - idx;
-            b = brow[d < db.len ? d : db.len - 1];
+          for (int e = 0; e < 4; ++e) {
+            const int idx = eb + nb * 8 + (lane & 3) * 2 + (e & 1);
+            const int64_t d = pi[e >> 1] - idx;
+            const float b = idx < NB ? brow[d < db.len ? d : db.len - 1] : bt[nb + 1 - (e >> 1)][e & 1];
+            s[nb][e] = fmaf(b, kLog2e, s[nb][e]);
           }
-          s[nb][e] = fmaf(b, kLog2e, s[nb][e]);
-        }
+      } else {
+#pragma unroll
+        for (int nb = 0; nb < kGmBK / 8; ++nb)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[nb][e] = fmaf(bt[nb + 1 - (e >> 1)][e & 1], kLog2e, s[nb][e]);
+      }
     }
     if (sl != 0.f) {
 #pragma unroll

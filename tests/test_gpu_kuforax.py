@@ -35,7 +35,7 @@ def i64(x):
 # =================================================================================================
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("heads,kvh,dim,rot,paired", [
-    (4, 2, 16, 8, False), (1, 1, 10, 10, False), (6, 3, 64, 16, False), (2, 1, 6, 0, False), (5, 1, 128, 128, False),
+    (4, 2, 16, 8, False), (1, 1, 10, 10, False), (9, 3, 64, 48, False), (2, 1, 6, 0, False), (5, 1, 128, 128, False),
     (3, 3, 7, 6, False), (32, 8, 128, 64, False), (4, 2, 64, 32, True), (2, 2, 10, 6, True)])
 def test_row_norm_before_the_rotation(dtype, heads, kvh, dim, rot, paired):
     """q and k as slices of one wider row: an RMS norm over all heads together with a weight per channel, rotation with a
@@ -129,7 +129,7 @@ def _route(z, corr, top, groups):
                                 keep_groups=groups[1] if groups else 1, group_top=1)
 
 
-@pytest.mark.parametrize("n,top,groups", [(8, 3, (4, 2)), (6, 4, (3, 2)), (14, 4, (2, 1)), (2, 1, None), (5, 5, None),
+@pytest.mark.parametrize("n,top,groups", [(8, 3, (4, 2)), (6, 4, (3, 2)), (16, 5, (2, 1)), (2, 1, None), (5, 5, None),
                                           (200, 8, (10, 4)), (9, 2, (9, 3)), (3, 2, (1, 1))])
 def test_routing_by_groups(n, top, groups):
     """Corrections pull the choice scores of half the tokens below zero; weights come from the scores alone."""
@@ -229,7 +229,7 @@ ATTN_CASES = [
     ("kept-beyond-a-tile", 4, 4, 128, 128, 30, 150, None),
     ("kept-one", 1, 1, 6, 4, 1, 1, None),
     ("bias", 4, 2, 16, 24, 21, 0, (12, 30)),
-    ("bias-tiles", 8, 4, 64, 64, 72, 0, (32, 120)),
+    ("bias-tiles", 10, 5, 64, 64, 77, 0, (28, 110)),
     ("bias-saturates", 4, 2, 64, 128, 130, 0, (16, 40)),
     ("bias-no-window", 6, 2, 128, 128, None, 0, (7, 50)),
     ("bias-one-row", 3, 1, 10, 6, None, 0, (1, 5)),
